@@ -33,7 +33,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 12
+#define B200_ABI_VERSION 13
 
 enum {
   B200_OK = 0,
@@ -47,7 +47,7 @@ enum {
 /* B200_INT8_WO is only valid as a GEMM `ab_dtype`: bf16 activations x int8 weights (weight-only quantisation) */
 enum { B200_BF16 = 0, B200_FP8_E4M3 = 1, B200_INT8 = 2, B200_F32 = 3, B200_INT8_WO = 4 };
 /* gate activations of a gated-linear unit, and how a router turns its chosen logits into weights */
-enum { B200_ACT_SWISH_CLAMPED = 0, B200_ACT_SILU = 1, B200_ACT_GELU_TANH = 2 };
+enum { B200_ACT_SWISH_CLAMPED = 0, B200_ACT_SILU = 1, B200_ACT_GELU_TANH = 2, B200_ACT_NONE = 3, B200_ACT_RELU2 = 4 };
 enum { B200_ROUTE_SIGMOID = 0, B200_ROUTE_SOFTMAX_TOP = 1, B200_ROUTE_SOFTMAX_RENORM = 2 };
 
 int b200_abi_version(void);
@@ -355,7 +355,7 @@ int b200_swa_sink_attn(const float* q, int ldq, const void* k_pool, const void* 
                        int64_t bt_stride, const int32_t* tok_row, const int32_t* tok_pos, const float* sink, float scale,
                        int window, void* out, int T, int H, int G, int D, int Dv, int v_pitch, int block_size, int chunk,
                        float softcap, const float* sigmoid_bias, int v_div, int out_f32, int splits, float* split_workspace,
-                       const void* pooled_k, const void* pooled_v, int pool, void* stream);
+                       const void* pooled_k, const void* pooled_v, int pool, int keep, void* stream);
 /* Means of the key / value blocks that the step completes: sequence s brings tokens [seq_start[s], seq_start[s+1]) at positions
  * seq_pos0[s].. (block-table row seq_slot[s]); for every block of `pool` positions whose last position is among them the block's
  * `pool` key and value rows are read back from the pools, summed in fp32, divided by `pool` and written to
@@ -374,9 +374,10 @@ int b200_swa_sink_attn_prefill(const float* q, int ldq, const void* k_pool, cons
                                int64_t bt_stride, const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_pos0,
                                int B, int max_new, const float* sink, float scale, int window, void* out, int H, int G, int D,
                                int Dv, int v_pitch, int block_size, int chunk, float softcap, const float* sigmoid_bias, int v_div,
-                               int out_f32, int split_p, const void* pooled_k, const void* pooled_v, int pool, void* stream);
+                               int out_f32, int split_p, const void* pooled_k, const void* pooled_v, int pool, int keep,
+                               void* stream);
 /* Prompt portions on the 5th-generation tensor cores (tcgen05, accumulators in tensor memory): same ragged step arguments as
- * b200_swa_sink_attn_prefill, no sink and no window.  Kernels exist for pages of 32 tokens and D = Dv = 64 or 128 (softmax,
+ * b200_swa_sink_attn_prefill, no sink; window 0 = none.  Kernels exist for pages of 32 tokens and D = Dv = 64 or 128 (softmax,
  * capped softmax, sigmoid weights) and, with v_div = 2, D = 32 or 64 with Dv = 64 or 128 (softmax); q rows must be 16-byte aligned.
  * b200_swa_sink_attn_prefill_tc_supported says whether a combination has one; the launch returns B200_ERR_UNSUPPORTED
  * otherwise.  num_blocks = pages of the pools. */
@@ -385,7 +386,7 @@ int b200_swa_sink_attn_prefill_tc(const float* q, int ldq, const void* k_pool, c
                                   const int32_t* block_table, int64_t bt_stride, const int32_t* seq_start,
                                   const int32_t* seq_slot, const int32_t* seq_pos0, int B, int max_new, float scale, void* out,
                                   int H, int G, int D, int Dv, int block_size, int chunk, float softcap,
-                                  const float* sigmoid_bias, int v_div, int out_f32, int split_p, void* stream);
+                                  const float* sigmoid_bias, int v_div, int out_f32, int split_p, int window, int keep, void* stream);
 /* The same attention for decode-sized steps on the tensor cores (bf16 pools with a value pool of its own; D and Dv multiples of
  * 16, Dv <= 256, else B200_ERR_UNSUPPORTED): the query heads of a kv head are the rows of one MMA tile, each key and value row
  * is fetched once for all of them.  Arguments as b200_swa_sink_attn (+ split_p as in the prompt kernel). */
@@ -393,14 +394,15 @@ int b200_swa_sink_attn_decode_tc(const float* q, int ldq, const void* k_pool, co
                                  int64_t bt_stride, const int32_t* tok_row, const int32_t* tok_pos, const float* sink, float scale,
                                  int window, void* out, int T, int H, int G, int D, int Dv, int v_pitch, int block_size, int chunk,
                                  float softcap, const float* sigmoid_bias, int v_div, int out_f32, int split_p, int splits,
-                                 float* split_workspace, const void* pooled_k, const void* pooled_v, int pool, void* stream);
+                                 float* split_workspace, const void* pooled_k, const void* pooled_v, int pool, int keep, void* stream);
 /* Merge of key splits: part fp32 [rows][splits][2 + Dv] = {maximum, denominator, unnormalised accumulator} per split ->
  * out [rows][Dv] (fp32 when out_f32, else out_dtype); sigmoid: plain sums, no denominator. */
 int b200_attn_split_merge(const float* part, int splits, int Dv, int sigmoid, int out_f32, int out_dtype, void* out, int64_t rows,
                           void* stream);
 /* Between the projections and the attention of layers that norm and rotate: fp32 rows `src` (pitch ld) hold q [H][D] at
  * q_col0, k [G][D] at k_col0, v [Gv][Dv] at v_col0.  q_norm / k_norm fp32 [H * D] / [G * D] (or NULL): RMS norm over the WHOLE
- * projection, times the weight.  The first rot_n columns of every q and k head turn by tok_pos[t]: pairs (i, i + rot_n / 2) when
+ * projection, times the weight; with head_norm each head is divided by its own RMS and the weights are fp32 [D], shared by the
+ * heads.  v_col0 may equal k_col0 (the values are the keys as projected).  The first rot_n columns of every q and k head turn by tok_pos[t]: pairs (i, i + rot_n / 2) when
  * rot_half, else (2i, 2i + 1); (u, v) -> (u cos - v sin, v cos + u sin), cos / sin fp32 tables [positions][rot_n / 2].
  * q -> q_out fp32 [T][H * D], head h times q_head_scale[h] when given (a per-head temperature of the scores);
  * k, v -> pools K [num_blocks][G][block_size][D], V [num_blocks][Gv][block_size][Dv] by slot. */
@@ -408,7 +410,7 @@ int b200_qk_norm_rope_kv_write(const float* src, int ld, int q_col0, int k_col0,
                                const float* k_norm, float eps, int rot_n, int rot_half, const float* cos_table,
                                const float* sin_table, const int32_t* tok_pos, const int64_t* slot_mapping, float* q_out,
                                void* k_pool, void* v_pool, int kv_dtype, int T, int H, int G, int Gv, int D, int Dv, int block_size,
-                               const float* q_head_scale, void* stream);
+                               const float* q_head_scale, int head_norm, void* stream);
 /* Router decision over fp32 logits [T] rows of pitch ld (+ bias fp32 [E] when given): the `top` largest (ties to the lower
  * index); weights = sigmoid of each chosen logit, no renormalisation (B200_ROUTE_SIGMOID), or the softmax over the chosen
  * logits only (B200_ROUTE_SOFTMAX_TOP), or the softmax over ALL experts with the chosen scores divided by their sum + 1e-20
@@ -502,6 +504,42 @@ int b200_gated_scan_prep(float* proj, int ld, int q_col0, int f_col0, int n, con
 int b200_gated_scan(const float* proj, int ld, int q_col0, int f_col0, int v_col0, float* state, const int32_t* seq_start,
                     const int32_t* seq_slot, const int32_t* seq_pos0, float* out, int B, int H, int D, int P, const int32_t* segs,
                     int num_segs, const int32_t* seq_seg0, float* seg_state, float* seg_decay, void* stream);
+/* Matrix memory (mLSTM), gates: raw gate columns i_col0 / f_col0 ([H] each) of the fp32 rows proj, plus biases fp32 [H];
+ * i = cap tanh(raw_i / cap), f = log sigmoid(cap tanh(raw_f / cap)), m_t = max(f + m_(t-1), i) with m_0 = 0 (m_state fp32
+ * [slots][H] carries it, read when seq_pos0 > 0);  coef fp32 [T][H][2] = (exp(f + m_(t-1) - m_t), exp(i - m_t)),
+ * floor_out fp32 [T][H] = exp(-m_t). */
+int b200_matrix_memory_gates(const float* proj, int ld, int i_col0, int f_col0, const float* i_bias, const float* f_bias, float cap,
+                             float* m_state, const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_pos0,
+                             float* coef, float* floor_out, int B, int H, void* stream);
+/* Matrix memory, scan: per head S_t = a S_(t-1) + b k_t v_t^T and n_t = a n_(t-1) + b k_t with (a, b) = coef;
+ * out fp32 [T][H * P] = S_t^T q_t, out_n fp32 [T][H] = n_t . q_t; q, k [H][D] and v [H][P] are the columns q_col0 / k_col0 / v_col0 of
+ * the fp32 rows proj.  state fp32 [slots][H][P + 1][D], the last column n.  Segments as in b200_gated_scan (scratch
+ * [num_segs][H][P + 1][D] and [num_segs][H][D]).  D <= 512, else B200_ERR_UNSUPPORTED. */
+int b200_matrix_memory_scan(const float* proj, int ld, int q_col0, int k_col0, int v_col0, const float* coef, float* state,
+                            const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_pos0, float* out, float* out_n,
+                            int B, int H, int D, int P, const int32_t* segs, int num_segs, const int32_t* seq_seg0,
+                            float* seg_state, float* seg_decay, void* stream);
+/* Matrix memory, output: u = scale o / (max(|scale nq|, floor) + 1e-6) per head, out = u / sqrt(mean_P(u^2) + eps) * w * sigmoid(gate);
+ * w fp32 [H * P], gate = columns gate_col0.. of fp32 rows (pitch ldg). */
+int b200_matrix_memory_out(const float* o, const float* nq, const float* floor_in, float scale, const float* gate, int ldg,
+                           int gate_col0, const float* w, float eps, void* out, int out_dtype, int T, int H, int P, void* stream);
+/* Selective state-space scan with a step size per channel: S[c][n] <- exp(dt_c A[c][n]) S[c][n] + dt_c x_c B_n,
+ * y_c = sum_n S[c][n] C_n + d_skip_c x_c, out = y silu(z) (z NULL: y).  x, out [T][C] in x_dtype; dt = softplus(dt_raw + dt_bias);
+ * B, C = columns b_col0 / c_col0 ([N] each) of the fp32 rows bc; a_log2 fp32 [C][N] = A log2(e); state fp32 [slots][C][N], read when
+ * seq_pos0 > 0, written back for all.  num_segs > 0: segments as in b200_gated_scan, scratch seg_state fp32 [num_segs][C][N] and
+ * seg_dt fp32 [num_segs][C].  N <= 256, else B200_ERR_UNSUPPORTED. */
+int b200_selective_scan(const void* x, int x_dtype, const float* dt_raw, int ld_dt, const float* bc, int ld_bc, int b_col0, int c_col0,
+                        const float* z, int ld_z, const float* a_log2, const float* dt_bias, const float* d_skip, float* state,
+                        const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_pos0, void* out, int B, int C, int N,
+                        const int32_t* segs, int num_segs, const int32_t* seq_seg0, float* seg_state, float* seg_dt, void* stream);
+/* Post-norm residual step with a layer norm: u = alpha x + [vec +] c (N(y1) w1 + N(y2) w2), N = division by the row's RMS (y2 NULL:
+ * u = alpha x + [vec +] c y1, y1 may be NULL too);  x (when store_x) = out (when given) = (u - mean) / sqrt(var + eps) * w. */
+int b200_postln_residual(float* x, float alpha, const float* y1, int ld1, const float* w1, const float* y2, int ld2, const float* w2,
+                         float c, const float* vec, const float* w, float eps, int store_x, void* out, int out_dtype, int T, int W,
+                         void* stream);
+/* out [T][n] = act(columns [col0, col0 + n) of the fp32 rows in + bias), act = B200_ACT_NONE or B200_ACT_RELU2 (square of relu);
+ * bias fp32 [n] or NULL */
+int b200_bias_act(const float* in, int ld, int col0, int n, const float* bias, int act, void* out, int out_dtype, int T, void* stream);
 /* gate_up fp32 [T][2 ff] (gate first): out = act(gate) * up, act = B200_ACT_SILU or B200_ACT_GELU_TANH */
 int b200_glu(const float* gate_up, void* out, int out_dtype, int T, int ff, int act, void* stream);
 /* Gated delta rule, preparation: qkv fp32 rows [q: G*D | k: G*D | v: H*P] (pitch ldc) are the convolved activations; q and k

@@ -12,9 +12,10 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libb200_paged.so")
 
 OK = 0
-ABI_VERSION = 12
+ABI_VERSION = 13
 BF16, FP8_E4M3, INT8, F32 = 0, 1, 2, 3
 ACT_SWISH_CLAMPED, ACT_SILU, ACT_GELU_TANH = 0, 1, 2   # gate activation of a gated-linear unit
+ACT_NONE, ACT_RELU2 = 3, 4   # plain activation behind a bias: identity, square of relu
 ROUTE_SIGMOID, ROUTE_SOFTMAX_TOP, ROUTE_SOFTMAX_RENORM = 0, 1, 2   # router weights: sigmoid of each chosen logit | softmax over
 # the chosen | softmax over all experts, the chosen scores divided by their sum
 
@@ -81,18 +82,18 @@ SIGNATURES = {
     "b200_kv_write_vmix": (_i, [_p, _i, _i, _i, _p, _f, _i, _p, _p, _i, _p, _i, _i, _i, _i, _i, _p]),
     "b200_causal_conv": (_i, [_p, _i, _i, _p, _p, _p, _i, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _p]),
     "b200_swa_sink_attn": (_i, [_p, _i, _p, _p, _i, _p, _i64, _p, _p, _p, _f, _i, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _i, _i,
-                                _i, _p, _p, _p, _i, _p]),
+                                _i, _p, _p, _p, _i, _i, _p]),
     "b200_kv_pool_mean": (_i, [_p, _p, _p, _p, _i, _p, _i64, _p, _p, _p, _i, _i, _i, _i, _i, _i, _i, _i, _p]),
     "b200_swa_sink_attn_prefill": (_i, [_p, _i, _p, _p, _p, _i64, _p, _p, _p, _i, _i, _p, _f, _i, _p, _i, _i, _i, _i, _i, _i, _i, _f,
-                                        _p, _i, _i, _i, _p, _p, _i, _p]),
+                                        _p, _i, _i, _i, _p, _p, _i, _i, _p]),
     "b200_swa_sink_attn_prefill_tc_supported": (_i, [_i, _i, _i, _i, _i, _i]),
     "b200_swa_sink_attn_prefill_tc": (_i, [_p, _i, _p, _p, _i, _p, _i64, _p, _p, _p, _i, _i, _f, _p, _i, _i, _i, _i, _i, _i, _f, _p, _i,
-                                           _i, _i, _p]),
+                                           _i, _i, _i, _i, _p]),
     "b200_swa_sink_attn_decode_tc": (_i, [_p, _i, _p, _p, _p, _i64, _p, _p, _p, _f, _i, _p, _i, _i, _i, _i, _i, _i, _i, _i, _f, _p, _i,
-                                          _i, _i, _i, _p, _p, _p, _i, _p]),
+                                          _i, _i, _i, _p, _p, _p, _i, _i, _p]),
     "b200_attn_split_merge": (_i, [_p, _i, _i, _i, _i, _i, _p, _i64, _p]),
     "b200_qk_norm_rope_kv_write": (_i, [_p, _i, _i, _i, _i, _p, _p, _f, _i, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i,
-                                        _i, _i, _p, _p]),
+                                        _i, _i, _p, _i, _p]),
     "b200_moe_topk": (_i, [_p, _i, _p, _i, _p, _p, _i, _i, _i, _p]),
     "b200_moe_tile_rows": (_i, []),
     "b200_moe_gather_scale": (_i, [_p, _i, _p, _i, _i, _p, _p, _i, _p, _i, _p]),
@@ -114,6 +115,14 @@ SIGNATURES = {
     "b200_scaled_add_rmsnorm2": (_i, [_p, _p, _i, _f, _p, _i, _f, _p, _i, _p, _f, _p, _p, _p, _p, _p, _p, _f, _i, _i, _i, _p]),
     "b200_gated_scan_prep": (_i, [_p, _i, _i, _i, _i, _p, _p, _i, _p]),
     "b200_gated_scan": (_i, [_p, _i, _i, _i, _i, _p, _p, _p, _p, _p, _i, _i, _i, _i, _p, _i, _p, _p, _p, _p]),
+    # post-layer-norm decoders: selective scan, matrix memory, layer-norm residual step, bias + activation
+    "b200_matrix_memory_gates": (_i, [_p, _i, _i, _i, _p, _p, _f, _p, _p, _p, _p, _p, _p, _i, _i, _p]),
+    "b200_matrix_memory_scan": (_i, [_p, _i, _i, _i, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _p, _i, _p, _p, _p, _p]),
+    "b200_matrix_memory_out": (_i, [_p, _p, _p, _f, _p, _i, _i, _p, _f, _p, _i, _i, _i, _i, _p]),
+    "b200_selective_scan": (_i, [_p, _i, _p, _i, _p, _i, _i, _i, _p, _i, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _p, _i, _p, _p, _p,
+                                 _p]),
+    "b200_postln_residual": (_i, [_p, _f, _p, _i, _p, _p, _i, _p, _f, _p, _p, _f, _i, _p, _i, _i, _i, _p]),
+    "b200_bias_act": (_i, [_p, _i, _i, _i, _p, _i, _p, _i, _i, _p]),
     "b200_delta_prep": (_i, [_p, _i, _p, _i, _i, _i, _p, _p, _p, _p, _i, _i, _i, _i, _f, _f, _p]),
     "b200_delta_scan": (_i, [_p, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p]),
     "b200_latent_kv_write": (_i, [_p, _i, _i, _i, _i, _i, _p, _f, _p, _p, _p, _p, _p, _i, _i, _p]),

@@ -344,6 +344,147 @@ __global__ void scaled_add_rmsnorm2_kernel(float* __restrict__ x, const float* _
   }
 }
 
+// Post-norm residual step with a layer norm (no bias):
+//   u = alpha x[t] + [vec +] c (y1[t] / rms(y1[t]) * w1 + y2[t] / rms(y2[t]) * w2)          (branches with norms of their own: y2 given)
+//   u = alpha x[t] + [vec +] c y1[t]                                                        (one plain branch; y1 may be absent too)
+//   x[t] = out[t] = (u - mean(u)) / sqrt(mean((u - mean(u))^2) + eps) * w
+// One CTA per token; the row stays in shared memory (16-byte accesses when rows sit on the 16-byte grid, V = 4).  Every sum has a
+// fixed order, so a row does not depend on what else is in the batch.  x is written when store_x is set, out when given.
+template <typename OT, int V>
+__global__ void postln_residual_kernel(float* __restrict__ x, float alpha, const float* __restrict__ y1, int ld1,
+                                       const float* __restrict__ w1, const float* __restrict__ y2, int ld2, const float* __restrict__ w2,
+                                       float c, const float* __restrict__ vec, const float* __restrict__ w, float eps, int store_x,
+                                       OT* __restrict__ out, int W) {
+  griddep_launch();
+  griddep_wait();
+  extern __shared__ __align__(16) float row[];
+  __shared__ float red[2 * 33];
+  const int t = blockIdx.x, warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = (blockDim.x + 31) >> 5;
+  float* xr = x + (int64_t)t * W;
+  const float *r1 = y1 ? y1 + (int64_t)t * ld1 : nullptr, *r2 = y2 ? y2 + (int64_t)t * ld2 : nullptr;
+  struct Vec {
+    float v[V];
+  };
+  auto ld = [](const float* p) -> Vec {
+    Vec a;
+    if constexpr (V == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(p);
+      a.v[0] = f.x, a.v[1] = f.y, a.v[2] = f.z, a.v[3] = f.w;
+    } else {
+      a.v[0] = *p;
+    }
+    return a;
+  };
+  auto st = [](float* p, const Vec& a) {
+    if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(a.v[0], a.v[1], a.v[2], a.v[3]);
+    else *p = a.v[0];
+  };
+  float i1 = c, i2 = c;
+  if (r2) {  // both branches' sums of squares in one round
+    float a = 0.f, b = 0.f;
+    for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+      const Vec u = ld(r1 + i), v = ld(r2 + i);
+#pragma unroll
+      for (int k = 0; k < V; ++k) a += u.v[k] * u.v[k], b += v.v[k] * v.v[k];
+    }
+    a = warp_sum(a), b = warp_sum(b);
+    if (lane == 0) red[warp] = a, red[33 + warp] = b;
+    __syncthreads();
+    if (warp < 2) {
+      const float s = warp_sum(lane < nw ? red[33 * warp + lane] : 0.f);
+      __syncwarp();
+      if (lane == 0) red[33 * warp + 32] = s;
+    }
+    __syncthreads();
+    i1 = c / sqrtf(red[32] / (float)W + eps);
+    i2 = c / sqrtf(red[33 + 32] / (float)W + eps);
+    __syncthreads();
+  }
+  float sum = 0.f;
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+    Vec u = ld(xr + i);
+#pragma unroll
+    for (int k = 0; k < V; ++k) u.v[k] *= alpha;
+    if (r1) {
+      const Vec a = ld(r1 + i);
+      if (r2) {
+        const Vec b = ld(r2 + i), wa = ld(w1 + i), wb = ld(w2 + i);
+#pragma unroll
+        for (int k = 0; k < V; ++k) u.v[k] += a.v[k] * i1 * wa.v[k] + b.v[k] * i2 * wb.v[k];
+      } else {
+#pragma unroll
+        for (int k = 0; k < V; ++k) u.v[k] += c * a.v[k];
+      }
+    }
+    if (vec) {
+      const Vec b = ld(vec + i);
+#pragma unroll
+      for (int k = 0; k < V; ++k) u.v[k] += b.v[k];
+    }
+    st(row + i, u);
+#pragma unroll
+    for (int k = 0; k < V; ++k) sum += u.v[k];
+  }
+  const float mean = block_sum(sum, red) / (float)W;
+  float ss = 0.f;
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+    const Vec u = ld(row + i);
+#pragma unroll
+    for (int k = 0; k < V; ++k) ss += (u.v[k] - mean) * (u.v[k] - mean);
+  }
+  const float inv = 1.0f / sqrtf(block_sum(ss, red) / (float)W + eps);
+  for (int i = threadIdx.x * V; i < W; i += blockDim.x * V) {
+    Vec u = ld(row + i);
+    const Vec g = ld(w + i);
+#pragma unroll
+    for (int k = 0; k < V; ++k) u.v[k] = (u.v[k] - mean) * inv * g.v[k];
+    if (store_x) st(xr + i, u);
+    if (out) {
+      OT* o = out + (int64_t)t * W + i;
+      if constexpr (V == 4 && sizeof(OT) == 2) {
+        *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16(u.v[0], u.v[1]), pack_bf16(u.v[2], u.v[3]));
+      } else if constexpr (V == 4) {
+        *reinterpret_cast<float4*>(o) = make_float4(u.v[0], u.v[1], u.v[2], u.v[3]);
+      } else {
+        stf(out, (int64_t)t * W + i, u.v[0]);
+      }
+    }
+  }
+}
+
+// out[t][i] = act(in[t][col0 + i] + bias[i]), act = identity or the square of relu; V columns per thread
+template <typename OT, int V>
+__global__ void bias_act_kernel(const float* __restrict__ in, int ld, int col0, int n, const float* __restrict__ bias, int act,
+                                OT* __restrict__ out, int64_t total) {
+  griddep_launch();
+  griddep_wait();
+  const int nv = n / V;
+  for (int64_t idx = (int64_t)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (int64_t)gridDim.x * blockDim.x) {
+    const int64_t t = idx / nv;
+    const int i = (int)(idx - t * nv) * V;
+    const float* p = in + t * ld + col0 + i;
+    float v[V];
+    if constexpr (V == 4) {
+      const float4 f = *reinterpret_cast<const float4*>(p);
+      v[0] = f.x, v[1] = f.y, v[2] = f.z, v[3] = f.w;
+    } else {
+      v[0] = *p;
+    }
+#pragma unroll
+    for (int k = 0; k < V; ++k) {
+      if (bias) v[k] += bias[i + k];
+      if (act == B200_ACT_RELU2) v[k] = v[k] > 0.f ? v[k] * v[k] : 0.f;
+    }
+    OT* o = out + t * n + i;
+    if constexpr (V == 4 && sizeof(OT) == 2) {
+      *reinterpret_cast<uint2*>(o) = make_uint2(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]));
+    } else {
+#pragma unroll
+      for (int k = 0; k < V; ++k) stf(o, k, v[k]);
+    }
+  }
+}
+
 template <typename OT>
 __global__ void glu_kernel(const float* __restrict__ gu, OT* __restrict__ out, int ff, int act, int64_t total) {
   griddep_launch();
@@ -436,6 +577,49 @@ int b200_scaled_add_rmsnorm2(float* x, const float* y1, int ld1, float c1, const
     B200_CUDA_OK(launch_kernel(scaled_add_rmsnorm2_kernel<OT>, dim3(T), dim3(W >= 1024 ? 256 : 128), smem, (cudaStream_t)stream, x,
                                y1, ld1, c1, y2, ld2, c2, y3, nsum, y3_weight, c3, add_rows, add_vec, w1, (OT*)out1, w2, (OT*)out2,
                                eps, W));
+  });
+  return B200_OK;
+}
+
+int b200_postln_residual(float* x, float alpha, const float* y1, int ld1, const float* w1, const float* y2, int ld2, const float* w2,
+                         float c, const float* vec, const float* w, float eps, int store_x, void* out, int out_dtype, int T, int W,
+                         void* stream) {
+  B200_REQUIRE(x && w && (!y2 || (y1 && w1 && w2)), "postln_residual: null pointer");
+  B200_REQUIRE(W >= 1 && (size_t)W * 4 <= 200 * 1024, "postln_residual: rows of %d do not fit shared memory", W);
+  if (T <= 0) return B200_OK;
+  const size_t smem = (size_t)W * 4;
+  auto a16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
+  const bool v4 = W % 4 == 0 && ld1 % 4 == 0 && ld2 % 4 == 0 && a16(x) && a16(y1) && a16(y2) && a16(w1) && a16(w2) && a16(vec) &&
+                  a16(w) && a16(out);
+  const int per = v4 ? W / 4 : W, threads = per > 512 ? 512 : per > 256 ? 256 : per > 128 ? 128 : 64;
+#define POSTLN(V)                                                                                                                  \
+  B200_DISPATCH_ELEM(out_dtype, OT, {                                                                                              \
+    if (smem > 48 * 1024)                                                                                                          \
+      B200_CUDA_OK(cudaFuncSetAttribute(postln_residual_kernel<OT, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));   \
+    B200_CUDA_OK(launch_kernel(postln_residual_kernel<OT, V>, dim3(T), dim3(threads), smem, (cudaStream_t)stream, x, alpha, y1,    \
+                               ld1, w1, y2, ld2, w2, c, vec, w, eps, store_x, (OT*)out, W));                                       \
+  })
+  if (v4) POSTLN(4);
+  else POSTLN(1);
+#undef POSTLN
+  return B200_OK;
+}
+
+int b200_bias_act(const float* in, int ld, int col0, int n, const float* bias, int act, void* out, int out_dtype, int T, void* stream) {
+  B200_REQUIRE(in && out && n >= 1 && col0 >= 0, "bias_act: null pointer or bad shape");
+  B200_REQUIRE(act == B200_ACT_NONE || act == B200_ACT_RELU2, "bias_act: activation %d", act);
+  if (T <= 0) return B200_OK;
+  const bool v4 = n % 4 == 0 && ld % 4 == 0 && col0 % 4 == 0 && ((uintptr_t)in & 15) == 0 && ((uintptr_t)out & 15) == 0;
+  const int64_t total = (int64_t)T * (v4 ? n / 4 : n);
+  int64_t blocks = (total + 255) / 256;
+  blocks = blocks > 148 * 16 ? 148 * 16 : blocks;
+  B200_DISPATCH_ELEM(out_dtype, OT, {
+    if (v4)
+      B200_CUDA_OK(launch_kernel(bias_act_kernel<OT, 4>, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, in, ld, col0, n,
+                                 bias, act, (OT*)out, total));
+    else
+      B200_CUDA_OK(launch_kernel(bias_act_kernel<OT, 1>, dim3((unsigned)blocks), dim3(256), 0, (cudaStream_t)stream, in, ld, col0, n,
+                                 bias, act, (OT*)out, total));
   });
   return B200_OK;
 }

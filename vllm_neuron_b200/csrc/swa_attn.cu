@@ -11,9 +11,9 @@
 //     Variants of the same kernel, all parameters: keys confined to the query's CHUNK of positions (counted from position 0),
 //     a soft cap on the scaled score (cap tanh(s / cap)), SIGMOID weights sigmoid(s + bias[head]) that are not normalised
 //     over the keys (then no sink, no maximum, no denominator), several key heads sharing one value head (v_div: two score
-//     maps over the same values), and fp32 output rows;
+//     maps over the same values), the first `keep` tokens of the sequence visible beside the window, and fp32 output rows;
 //   * qk_norm_rope_kv_write: the step between the projections (or their short convolutions) and the attention of layers
-//     that norm and rotate: an optional RMS norm over the WHOLE q (and k) projection, rotary positions from cos / sin tables
+//     that norm and rotate: an optional RMS norm over the WHOLE q (and k) projection or over each head, rotary positions from cos / sin tables
 //     on the leading columns of every head (pairs (i, i + n/2) or (2i, 2i + 1)), q to an fp32 buffer, k and v into the pools.
 // Pools: K [num_blocks][G][block_size][D], V [num_blocks][G][block_size][v_pitch] with values in the first Dv columns of a
 // row (v_pitch = Dv for a pool of its own; a value pool may alias the key pool, values = the leading columns of the key
@@ -48,8 +48,23 @@ __global__ void kv_write_vmix_kernel(const float* __restrict__ qkv, int ld, int 
   }
 }
 
-// One CTA per token.  src fp32 rows hold q [H][D] at q_col0, k [G][D] at k_col0 and v [Gv][Dv] at v_col0.  q and k are
-// (optionally) divided by the RMS of their whole projection and multiplied by a weight per column, then the first rot_n
+// 1 / rms of every q head (inv[0 .. H)) and k head (inv[H .. H + G)), a warp per head; a side without a norm is left out
+__device__ __forceinline__ void head_inverse_rms(const float* row, int q_col0, int k_col0, bool q_norm, bool k_norm, int H, int G,
+                                                 int D, float eps, float* inv) {
+  const int lane = threadIdx.x & 31;
+  for (int i = threadIdx.x >> 5; i < H + G; i += blockDim.x >> 5) {
+    if (!(i < H ? q_norm : k_norm)) continue;
+    const float* r = row + (i < H ? q_col0 + i * D : k_col0 + (i - H) * D);
+    float ss = 0.f;
+    for (int d = lane; d < D; d += 32) ss += r[d] * r[d];
+    ss = warp_sum(ss);
+    if (lane == 0) inv[i] = 1.0f / sqrtf(ss / (float)D + eps);
+  }
+}
+
+// One CTA per token.  src fp32 rows hold q [H][D] at q_col0, k [G][D] at k_col0 and v [Gv][Dv] at v_col0 (v_col0 may equal
+// k_col0: the values are then the keys as projected).  q and k are (optionally) divided by the RMS of their whole projection and
+// multiplied by a weight per column -- or, with head_norm, each head by its own RMS and a weight [D] that the heads share --, then the first rot_n
 // columns of every head turn by the token's position: column pairs (i, i + rot_n / 2) when rot_half, else (2i, 2i + 1); a pair
 // (u, v) becomes (u cos - v sin, v cos + u sin) with cos / sin from fp32 tables [positions][rot_n / 2] (any frequency
 // scaling and magnitude factor live in the tables).  q goes to q_out fp32 [T][H * D]; k and v to the pools by slot.
@@ -60,15 +75,19 @@ __global__ void qk_norm_rope_kv_write_kernel(const float* __restrict__ src, int 
                                              const float* __restrict__ sin_t, const int32_t* __restrict__ tok_pos,
                                              const int64_t* __restrict__ slots, float* __restrict__ q_out, KT* __restrict__ k_pool,
                                              KT* __restrict__ v_pool, int H, int G, int Gv, int D, int Dv, int bs,
-                                             const float* __restrict__ q_head_scale) {
+                                             const float* __restrict__ q_head_scale, int head_norm) {
   griddep_launch();
   griddep_wait();
+  extern __shared__ float inv_h[];  // head_norm: [H + G]
   __shared__ float red[2][33];
   const int t = blockIdx.x;
   const float* row = src + (int64_t)t * ld;
   const int nq = H * D, nk = G * D;
   float inv_q = 1.0f, inv_k = 1.0f;
-  if (q_norm || k_norm) {  // sums of squares over the whole projections
+  if (head_norm) {
+    head_inverse_rms(row, q_col0, k_col0, q_norm != nullptr, k_norm != nullptr, H, G, D, eps, inv_h);
+    __syncthreads();
+  } else if (q_norm || k_norm) {  // sums of squares over the whole projections
     float sq = 0.f, sk = 0.f;
     if (q_norm)
       for (int i = threadIdx.x; i < nq; i += blockDim.x) sq += row[q_col0 + i] * row[q_col0 + i];
@@ -104,6 +123,10 @@ __global__ void qk_norm_rope_kv_write_kernel(const float* __restrict__ src, int 
   // the value of column i of a projection after its norm
   auto turned = [&](int col0, const float* nw, float inv, int i) -> float {
     const int d = i % D;
+    if (head_norm && nw) {
+      inv = inv_h[(col0 == q_col0 ? 0 : H) + i / D];
+      nw -= i - d;  // the weight is per column of a head
+    }
     const float u = row[col0 + i] * (nw ? inv * nw[i] : 1.0f);
     if (d >= rot_n) return u;
     int partner, idx;
@@ -143,16 +166,20 @@ __global__ void qk_norm_rope_kv_write_vec_kernel(const float* __restrict__ src, 
                                                  const float* __restrict__ sin_t, const int32_t* __restrict__ tok_pos,
                                                  const int64_t* __restrict__ slots, float* __restrict__ q_out,
                                                  KT* __restrict__ k_pool, KT* __restrict__ v_pool, int H, int G, int Gv, int D, int Dv,
-                                                 int bs, const float* __restrict__ q_head_scale) {
+                                                 int bs, const float* __restrict__ q_head_scale, int head_norm) {
   griddep_launch();
   griddep_wait();
+  extern __shared__ float inv_h[];  // head_norm: [H + G]
   __shared__ float red[2][33];
   const int t = blockIdx.x;
   const float* row = src + (int64_t)t * ld;
   const int nq = H * D, nk = G * D;
   auto ld4 = [](const float* p) { return *reinterpret_cast<const float4*>(p); };
   float inv_q = 1.0f, inv_k = 1.0f;
-  if (q_norm || k_norm) {
+  if (head_norm) {
+    head_inverse_rms(row, q_col0, k_col0, q_norm != nullptr, k_norm != nullptr, H, G, D, eps, inv_h);
+    __syncthreads();
+  } else if (q_norm || k_norm) {
     float sq = 0.f, sk = 0.f;
     if (q_norm)
       for (int i = threadIdx.x * 4; i < nq; i += blockDim.x * 4) {
@@ -195,6 +222,11 @@ __global__ void qk_norm_rope_kv_write_vec_kernel(const float* __restrict__ src, 
   auto normed = [&](int col0, const float* nw, float inv, int i) -> float4 {
     float4 u = ld4(row + col0 + i);
     if (nw) {
+      if (head_norm) {
+        const int hd = i / D;
+        inv = inv_h[(col0 == q_col0 ? 0 : H) + hd];
+        nw -= hd * D;  // the weight is per column of a head
+      }
       const float4 w = ld4(nw + i);
       u.x *= inv * w.x, u.y *= inv * w.y, u.z *= inv * w.z, u.w *= inv * w.w;
     }
@@ -420,7 +452,7 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
                          const int32_t* __restrict__ tok_pos, const float* __restrict__ sink, float scale, int window,
                          void* __restrict__ out, int T, int H, int G, int D, int Dv, int bs, int v_pitch, int chunk, float softcap,
                          const float* __restrict__ sig_bias, int v_div, int out_f32, float* __restrict__ part,
-                         const KT* __restrict__ pk_pool, const KT* __restrict__ pv_pool, int pool, int ppb) {
+                         const KT* __restrict__ pk_pool, const KT* __restrict__ pv_pool, int pool, int ppb, int keep) {
   griddep_launch();
   griddep_wait();
   extern __shared__ __align__(16) float sm_att[];
@@ -457,14 +489,15 @@ __global__ void __launch_bounds__(ATT_WARPS * 32)
     for (int c = 0; c < MAXC; ++c) acc[qh][c] = make_float2(0.f, 0.f);
   }
   // pooled blocks: block b (positions b pool .. b pool + pool - 1) is seen as one key / value once it lies wholly before the
-  // window, b pool + pool - 1 <= pos - window; its row sits in the page of its last position.  The tile list is the pooled
-  // entries (32 per tile) followed by the window's keys.
-  const int nb = pool > 0 && pos - window + 1 > 0 ? (pos - window + 1) / pool : 0;
+  // window, b pool + pool - 1 <= pos - window; its row sits in the page of its last position.  Kept tokens (keep > 0, no
+  // pooled blocks): positions 0 .. keep - 1 that lie before the window.  The tile list is these early entries (32 per tile)
+  // followed by the window's keys.
+  const int nb = pool > 0 ? (pos - window + 1 > 0 ? (pos - window + 1) / pool : 0) : min(keep, lo);
   const int npt = (nb + 31) >> 5, ntt = ((pos - lo) >> 5) + 1;
   for (int ti = warp + ATT_WARPS * split; ti < npt + ntt; ti += ATT_WARPS * splits) {
-    const bool pooled = ti < npt;
-    const int j = pooled ? ti * 32 + lane : lo + (ti - npt) * 32 + lane;  // pooled block, or key position
-    const bool valid = pooled ? j < nb : j <= pos;
+    const bool early = ti < npt, pooled = early && pool > 0;
+    const int j = early ? ti * 32 + lane : lo + (ti - npt) * 32 + lane;  // pooled block, or key position
+    const bool valid = early ? j < nb : j <= pos;
     const KT* vrow = v_pool;  // lanes past the last key: row 0 of the pool (the null page, finite values) with weight 0
     float p[QH];
 #pragma unroll
@@ -619,12 +652,15 @@ int b200_qk_norm_rope_kv_write(const float* src, int ld, int q_col0, int k_col0,
                                const float* k_norm, float eps, int rot_n, int rot_half, const float* cos_table,
                                const float* sin_table, const int32_t* tok_pos, const int64_t* slot_mapping, float* q_out,
                                void* k_pool, void* v_pool, int kv_dtype, int T, int H, int G, int Gv, int D, int Dv, int block_size,
-                               const float* q_head_scale, void* stream) {
+                               const float* q_head_scale, int head_norm, void* stream) {
+  B200_REQUIRE(H + G <= 12000, "qk_norm_rope_kv_write: %d heads", H + G);
+  B200_REQUIRE(!head_norm || q_col0 != k_col0, "qk_norm_rope_kv_write: q and k share their columns");
   B200_REQUIRE(src && tok_pos && slot_mapping && q_out && k_pool && v_pool, "qk_norm_rope_kv_write: null pointer");
   B200_REQUIRE(rot_n >= 0 && rot_n <= D && rot_n % 2 == 0 && (rot_n == 0 || (cos_table && sin_table)),
                "qk_norm_rope_kv_write: %d rotating columns in heads of %d", rot_n, D);
   B200_REQUIRE(H >= 1 && G >= 1 && Gv >= 1 && D >= 1 && Dv >= 1, "qk_norm_rope_kv_write: bad shape");
   if (T <= 0) return B200_OK;
+  const size_t smem = head_norm ? (size_t)(H + G) * 4 : 0;
   auto a16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
   const bool vec = D % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && q_col0 % 4 == 0 && k_col0 % 4 == 0 && v_col0 % 4 == 0 &&
                    rot_n % (rot_half ? 8 : 4) == 0 && a16(src) && a16(q_out) && a16(k_pool) && a16(v_pool) && a16(q_norm) &&
@@ -633,17 +669,17 @@ int b200_qk_norm_rope_kv_write(const float* src, int ld, int q_col0, int k_col0,
     const int cols = H * D > G * D ? H * D : G * D;
     const int threads = cols >= 1024 ? 256 : cols >= 512 ? 128 : 64;
     B200_DISPATCH_ELEM(kv_dtype, KT,
-                       B200_CUDA_OK(launch_kernel(qk_norm_rope_kv_write_vec_kernel<KT>, dim3(T), dim3(threads), 0, (cudaStream_t)stream,
+                       B200_CUDA_OK(launch_kernel(qk_norm_rope_kv_write_vec_kernel<KT>, dim3(T), dim3(threads), smem, (cudaStream_t)stream,
                                                   src, ld, q_col0, k_col0, v_col0, q_norm, k_norm, eps, rot_n, rot_half, cos_table,
                                                   sin_table, tok_pos, slot_mapping, q_out, (KT*)k_pool, (KT*)v_pool, H, G, Gv, D, Dv,
-                                                  block_size, q_head_scale)));
+                                                  block_size, q_head_scale, head_norm)));
     return B200_OK;
   }
   B200_DISPATCH_ELEM(kv_dtype, KT,
-                     B200_CUDA_OK(launch_kernel(qk_norm_rope_kv_write_kernel<KT>, dim3(T), dim3(256), 0, (cudaStream_t)stream, src, ld,
+                     B200_CUDA_OK(launch_kernel(qk_norm_rope_kv_write_kernel<KT>, dim3(T), dim3(256), smem, (cudaStream_t)stream, src, ld,
                                                 q_col0, k_col0, v_col0, q_norm, k_norm, eps, rot_n, rot_half, cos_table, sin_table,
                                                 tok_pos, slot_mapping, q_out, (KT*)k_pool, (KT*)v_pool, H, G, Gv, D, Dv, block_size,
-                                                q_head_scale)));
+                                                q_head_scale, head_norm)));
   return B200_OK;
 }
 
@@ -665,7 +701,8 @@ int b200_swa_sink_attn(const float* q, int ldq, const void* k_pool, const void* 
                        int64_t bt_stride, const int32_t* tok_row, const int32_t* tok_pos, const float* sink, float scale,
                        int window, void* out, int T, int H, int G, int D, int Dv, int v_pitch, int block_size, int chunk,
                        float softcap, const float* sigmoid_bias, int v_div, int out_f32, int splits, float* split_workspace,
-                       const void* pooled_k, const void* pooled_v, int pool, void* stream) {
+                       const void* pooled_k, const void* pooled_v, int pool, int keep, void* stream) {
+  B200_REQUIRE(keep >= 0 && (keep == 0 || pool == 0), "swa_sink_attn: %d kept tokens beside pooled blocks", keep);
   B200_REQUIRE(q && k_pool && v_pool && block_table && tok_row && tok_pos && out, "swa_sink_attn: null pointer");
   B200_REQUIRE(pool >= 0 && (pool == 0 || (pooled_k && pooled_v && v_pool != k_pool)), "swa_sink_attn: blocks of %d need pooled pools", pool);
   const int ppb = pool > 0 ? (block_size + pool - 1) / pool : 0;
@@ -694,7 +731,7 @@ int b200_swa_sink_attn(const float* q, int ldq, const void* k_pool, const void* 
     B200_CUDA_OK(launch_kernel(swa_sink_attn_kernel<KT, MC, QH>, grid, dim3(ATT_WARPS * 32), smem, st, q, ldq,               \
                                (const KT*)k_pool, (const KT*)v_pool, block_table, bt_stride, tok_row, tok_pos, sink, scale, \
                                window, out, T, H, G, D, Dv, block_size, v_pitch, chunk, softcap, sigmoid_bias, v_div, out_f32,       \
-                               split_workspace, (const KT*)pooled_k, (const KT*)pooled_v, pool, ppb));                      \
+                               split_workspace, (const KT*)pooled_k, (const KT*)pooled_v, pool, ppb, keep));                      \
   } while (0)
 #define ATT_LAUNCH(MC)                \
   do {                                \

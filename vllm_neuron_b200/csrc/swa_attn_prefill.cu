@@ -34,7 +34,8 @@ __global__ void __launch_bounds__(PF_THREADS, DV16M <= 8 ? 512 / PF_THREADS : 25
                             const int32_t* __restrict__ seq_pos0, const float* __restrict__ sink, float scale, int window,
                             void* __restrict__ out, int H, int G, int D, int Dv, int bs, int v_pitch, int chunk, float softcap,
                             const float* __restrict__ sig_bias, int v_div, int out_f32, int split_p, int bs_shift,
-                            const __nv_bfloat16* __restrict__ pk_pool, const __nv_bfloat16* __restrict__ pv_pool, int pool, int ppb) {
+                            const __nv_bfloat16* __restrict__ pk_pool, const __nv_bfloat16* __restrict__ pv_pool, int pool, int ppb,
+                            int keep) {
   griddep_wait();
   // the last rows of a portion see the most keys: their tiles are launched first, so the longest CTAs do not form the tail
   const int sq = blockIdx.z, h = blockIdx.y, i0 = (gridDim.x - 1 - blockIdx.x) * PF_ROWS;
@@ -94,17 +95,18 @@ __global__ void __launch_bounds__(PF_THREADS, DV16M <= 8 ? 512 / PF_THREADS : 25
   // Pooled blocks (pool > 0): block b of `pool` positions is one key / value for the rows that have it wholly before their
   // window, b pool + pool - 1 <= position - window; its row sits in the pooled pools, in the page of the block's last position.
   // The CTA's tile list is the pooled entries its LAST row sees (32 per tile), then the key positions as before; tile `it`
-  // of the list is pooled while it < npt.
-  const int nb_max = pool > 0 && j_hi - window + 1 > 0 ? (j_hi - window + 1) / pool : 0;
-  const int npt = (nb_max + PF_KEYS - 1) / PF_KEYS;
+  // of the list is pooled while it < npt.  Kept tokens (keep > 0, no pooled blocks): positions 0 .. keep - 1 stay visible; those
+  // before the first window tile form the early tiles instead (every row sees them), the others are let through by the mask.
   const int j_first = (j_lo / PF_KEYS) * PF_KEYS;
+  const int nb_max = pool > 0 ? (j_hi - window + 1 > 0 ? (j_hi - window + 1) / pool : 0) : min(keep, j_first);
+  const int npt = (nb_max + PF_KEYS - 1) / PF_KEYS;
   const int ntiles = npt + (j_hi - j_first) / PF_KEYS + 1;
   // the page of this thread's row in tile `it` (looked up one tile before the copies that need it are issued)
   auto page_of = [&](int it) -> int64_t {
     if (it < npt) {
       const int b = it * PF_KEYS + ir;
       if (b >= nb_max) return 0;
-      const int e = b * pool + pool - 1;
+      const int e = pool > 0 ? b * pool + pool - 1 : b;
       return bt[bs_shift >= 0 ? e >> bs_shift : e / bs];
     }
     const int j = j_first + (it - npt) * PF_KEYS + ir;
@@ -115,7 +117,7 @@ __global__ void __launch_bounds__(PF_THREADS, DV16M <= 8 ? 512 / PF_THREADS : 25
     if (it < ntiles) {
       const __nv_bfloat16 *kr, *vr;
       bool ok;
-      if (it < npt) {
+      if (it < npt && pool > 0) {
         const int b = it * PF_KEYS + ir;
         ok = b < nb_max;
         const int e = b * pool + pool - 1;
@@ -123,8 +125,8 @@ __global__ void __launch_bounds__(PF_THREADS, DV16M <= 8 ? 512 / PF_THREADS : 25
         kr = pk_pool + ((blk * G + g) * ppb + idx) * D;
         vr = pv_pool + ((blk * Gv + gv) * ppb + idx) * Dv;
       } else {
-        const int j = j_first + (it - npt) * PF_KEYS + ir;
-        ok = j <= j_hi;
+        const int j = it < npt ? it * PF_KEYS + ir : j_first + (it - npt) * PF_KEYS + ir;
+        ok = it < npt ? j < nb_max : j <= j_hi;
         const int off = ok ? (bs_shift >= 0 ? j & (bs - 1) : j % bs) : 0;
         kr = k_pool + ((blk * G + g) * bs + off) * D;
         vr = v_pool + ((blk * Gv + gv) * bs + off) * v_pitch;
@@ -173,7 +175,7 @@ __global__ void __launch_bounds__(PF_THREADS, DV16M <= 8 ? 512 / PF_THREADS : 25
     // first row, none before the lower bound of its last row; the bounds grow with the position) skips the per-element mask
     float mx_lo = -INFINITY, mx_hi = -INFINITY;
     // (a pooled tile: every block of it wholly before the window of the warp's first row)
-    const bool whole = ptile ? (j0 + PF_KEYS) * pool - 1 <= w_first - window : j0 + PF_KEYS - 1 <= w_first && j0 >= w_lb;
+    const bool whole = ptile ? (pool > 0 ? (j0 + PF_KEYS) * pool - 1 <= w_first - window : j0 + PF_KEYS <= nb_max) : j0 + PF_KEYS - 1 <= w_first && j0 >= w_lb;
     if (whole && !sig && softcap <= 0.f) {
 #pragma unroll
       for (int j = 0; j < PF_NT; ++j) {
@@ -189,8 +191,9 @@ __global__ void __launch_bounds__(PF_THREADS, DV16M <= 8 ? 512 / PF_THREADS : 25
           const int key = j0 + 8 * j + 2 * (lane & 3) + (c & 1);
           const bool hi = c >= 2;
           const int pos = hi ? p_hi : p_lo;
-          const bool seen = whole || ((hi ? ok_hi : ok_lo) && (ptile ? key * pool + pool - 1 <= pos - window
-                                                                            : key <= pos && key >= (hi ? lb_hi : lb_lo)));
+          const bool seen = whole || ((hi ? ok_hi : ok_lo) &&
+                                      (ptile ? (pool > 0 ? key * pool + pool - 1 <= pos - window : key < nb_max)
+                                             : key <= pos && (key >= (hi ? lb_hi : lb_lo) || key < keep)));
           float v = s[j][c] * scale;
           // tanh(x) = 1 - 2 / (1 + e^(2x)): absolute error ~1e-7, so the capped score is good to ~1e-7 of the cap
           if (softcap > 0.f) v = softcap * (1.0f - __fdividef(2.0f, 1.0f + __expf(2.0f * v * inv_cap)));
@@ -308,7 +311,7 @@ __global__ void __launch_bounds__(DT_WARPS * 32)
                               const float* __restrict__ sink, float scale, int window, void* __restrict__ out, int H, int G, int D,
                               int Dv, int bs, int v_pitch, int chunk, float softcap, const float* __restrict__ sig_bias, int v_div,
                               int out_f32, int split_p, float* __restrict__ part, const __nv_bfloat16* __restrict__ pk_pool,
-                              const __nv_bfloat16* __restrict__ pv_pool, int pool, int ppb) {
+                              const __nv_bfloat16* __restrict__ pv_pool, int pool, int ppb, int keep) {
   griddep_wait();
   extern __shared__ __align__(16) unsigned char dt_sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -378,14 +381,15 @@ __global__ void __launch_bounds__(DT_WARPS * 32)
     pc_src[sl] = key ? (gv * v_div + mp) * ppb * D + (c - mp * kch) * 8 : gv * ppb * Dv + (c - kcht) * 8;
   }
   // pooled blocks: block b of `pool` positions is one key / value once it lies wholly before the window,
-  // b pool + pool - 1 <= pos - window; the tile list is the pooled entries (32 per tile), then the window's keys
-  const int nb = pool > 0 && pos - window + 1 > 0 ? (pos - window + 1) / pool : 0;
+  // b pool + pool - 1 <= pos - window.  Kept tokens (keep > 0, no pooled blocks): positions 0 .. keep - 1 before the window.  The
+  // tile list is these early entries (32 per tile), then the window's keys
+  const int nb = pool > 0 ? (pos - window + 1 > 0 ? (pos - window + 1) / pool : 0) : min(keep, lo);
   const int npt = (nb + LDT_KEYS - 1) / LDT_KEYS, ntt = (pos - lo) / LDT_KEYS + 1;
   for (int ti = warp + DT_WARPS * split; ti < npt + ntt; ti += DT_WARPS * splits) {
     // ---- this warp's 32 key and value rows -> its buffer (rows past the token's position / the last seen block are zeros)
-    const bool ptile = ti < npt;
-    const int j0 = ptile ? ti * LDT_KEYS : lo + (ti - npt) * LDT_KEYS;  // first pooled block / first key position of the tile
-    const int j_end = ptile ? nb - 1 : pos;                            // last visible one
+    const bool early = ti < npt, ptile = early && pool > 0;
+    const int j0 = early ? ti * LDT_KEYS : lo + (ti - npt) * LDT_KEYS;  // first pooled block / first key position of the tile
+    const int j_end = early ? nb - 1 : pos;                            // last visible one
     const int jm = j0 + lane;
     int my_blk = -1, my_off = 0;
     if (jm <= j_end) {
@@ -569,7 +573,9 @@ int b200_swa_sink_attn_prefill(const float* q, int ldq, const void* k_pool, cons
                                int64_t bt_stride, const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_pos0,
                                int B, int max_new, const float* sink, float scale, int window, void* out, int H, int G, int D,
                                int Dv, int v_pitch, int block_size, int chunk, float softcap, const float* sigmoid_bias, int v_div,
-                               int out_f32, int split_p, const void* pooled_k, const void* pooled_v, int pool, void* stream) {
+                               int out_f32, int split_p, const void* pooled_k, const void* pooled_v, int pool, int keep,
+                               void* stream) {
+  B200_REQUIRE(keep >= 0 && (keep == 0 || pool == 0), "swa_sink_attn_prefill: %d kept tokens beside pooled blocks", keep);
   B200_REQUIRE(pool >= 0 && (pool == 0 || (pooled_k && pooled_v && v_pool != k_pool)), "swa_sink_attn_prefill: blocks of %d need pooled pools", pool);
   const int ppb = pool > 0 ? (block_size + pool - 1) / pool : 0;
   B200_REQUIRE(q && k_pool && v_pool && block_table && seq_start && seq_slot && seq_pos0 && out,
@@ -596,7 +602,7 @@ int b200_swa_sink_attn_prefill(const float* q, int ldq, const void* k_pool, cons
     B200_CUDA_OK(launch_kernel(swa_sink_prefill_kernel<M>, grid, dim3(PF_THREADS), smem, st, q, ldq, (const BT*)k_pool,              \
                                (const BT*)v_pool, block_table, bt_stride, seq_start, seq_slot, seq_pos0, sink, scale, window, \
                                out, H, G, D, Dv, block_size, v_pitch, chunk, softcap, sigmoid_bias, v_div, out_f32, split_p, bs_shift, \
-                               (const BT*)pooled_k, (const BT*)pooled_v, pool, ppb));                                         \
+                               (const BT*)pooled_k, (const BT*)pooled_v, pool, ppb, keep));                                         \
   } while (0)
   if (Dv <= 64) PF_LAUNCH(4);
   else if (Dv <= 128) PF_LAUNCH(8);
@@ -609,7 +615,9 @@ int b200_swa_sink_attn_decode_tc(const float* q, int ldq, const void* k_pool, co
                                  int64_t bt_stride, const int32_t* tok_row, const int32_t* tok_pos, const float* sink, float scale,
                                  int window, void* out, int T, int H, int G, int D, int Dv, int v_pitch, int block_size, int chunk,
                                  float softcap, const float* sigmoid_bias, int v_div, int out_f32, int split_p, int splits,
-                                 float* split_workspace, const void* pooled_k, const void* pooled_v, int pool, void* stream) {
+                                 float* split_workspace, const void* pooled_k, const void* pooled_v, int pool, int keep,
+                                 void* stream) {
+  B200_REQUIRE(keep >= 0 && (keep == 0 || pool == 0), "swa_sink_attn_decode_tc: %d kept tokens beside pooled blocks", keep);
   B200_REQUIRE(pool >= 0 && (pool == 0 || (pooled_k && pooled_v)), "swa_sink_attn_decode_tc: blocks of %d need pooled pools", pool);
   const int ppb = pool > 0 ? (block_size + pool - 1) / pool : 0;
   B200_REQUIRE(q && k_pool && v_pool && block_table && tok_row && tok_pos && out, "swa_sink_attn_decode_tc: null pointer");
@@ -637,7 +645,7 @@ int b200_swa_sink_attn_decode_tc(const float* q, int ldq, const void* k_pool, co
     B200_CUDA_OK(launch_kernel(swa_sink_decode_tc_kernel<M>, grid, dim3(DT_WARPS * 32), smem, st, q, ldq, (const BT*)k_pool,    \
                                (const BT*)v_pool, block_table, bt_stride, tok_row, tok_pos, sink, scale, window, out, H, G, D,  \
                                Dv, block_size, v_pitch, chunk, softcap, sigmoid_bias, v_div, out_f32, split_p,                  \
-                               split_workspace, (const BT*)pooled_k, (const BT*)pooled_v, pool, ppb));                          \
+                               split_workspace, (const BT*)pooled_k, (const BT*)pooled_v, pool, ppb, keep));                          \
   } while (0)
   if (Dv <= 64) DT_LAUNCH(4);
   else if (Dv <= 128) DT_LAUNCH(8);

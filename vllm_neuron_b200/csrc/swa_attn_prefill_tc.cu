@@ -1,14 +1,16 @@
 // Prompt attention of the hybrid family's rotating-attention layers on the 5th-generation tensor cores (tcgen05 + TMEM):
 // ragged batches of prompt portions over the paged K / V pools, with the layer variants as parameters.
 //
-//   out[r][h] = sum_k w(q[r][h] . K[k] * scale) V[k],   k <= pos(r), and k >= the start of pos(r)'s chunk when chunk > 0
+//   out[r][h] = sum_k w(q[r][h] . K[k] * scale) V[k],   k <= pos(r), k >= the start of pos(r)'s chunk when chunk > 0, and
+//   pos(r) - k < window or k < keep when window > 0 (a sliding window beside which the sequence's first tokens stay visible)
 //   w = softmax over the visible keys | softmax of cap * tanh(. / cap) | sigmoid(. + bias[h]) (not normalised)
 //
 // The pipeline is the one of paged_attn_prefill_tc.cu (two 128-row query tiles per CTA in tensor memory, S0 | S1 | O0 | O1,
 // K / V steps of 128 keys gathered page by page with TMA, one softmax thread per query row, lazy running maximum); what
 // differs:
 //   * one launch serves every sequence of the step (grid z; start row, position and block-table row come from the step's
-//     device arrays), and a tile starts at the key step that holds the first key of its first row's chunk;
+//     device arrays), and a tile starts at the key step that holds the first key of its first row's chunk or window (the key
+//     steps of the kept tokens, when they lie before it, come first);
 //   * q arrives as fp32 rows: the softmax warpgroups round it to bf16 and lay it into the 128-byte-swizzled operand
 //     layout themselves;
 //   * key size and value size are separate template parameters (keys of 32 columns are 64-byte rows under the 64B swizzle),
@@ -84,7 +86,7 @@ __global__ void __launch_bounds__(TP_THREADS, 1)
                           const float* __restrict__ q, int ldq, const int32_t* __restrict__ block_table, int64_t bt_stride,
                           const int32_t* __restrict__ seq_start, const int32_t* __restrict__ seq_slot,
                           const int32_t* __restrict__ seq_pos0, void* __restrict__ out, int H, int G, int chunk, float scale,
-                          float softcap, const float* __restrict__ sig_bias, int out_f32, int split_p, int ny_tiles) {
+                          float softcap, const float* __restrict__ sig_bias, int out_f32, int split_p, int ny_tiles, int window, int keep) {
   // q / k operand rows: pieces of 64 columns (128 bytes, 128B swizzle), or one piece of 32 columns (64 bytes, 64B swizzle)
   constexpr int KROW = DK >= 64 ? 128 : DK * 2;
   constexpr int NHK = DK >= 64 ? DK / 64 : 1, NHV = DV / 64;
@@ -126,9 +128,16 @@ __global__ void __launch_bounds__(TP_THREADS, 1)
   }
   const int q_hi = q0 + TP_BM < n_new ? q0 + TP_BM : n_new;
   const int kv_end = pos0 + q_hi;                                   // keys [0, kv_end) are visible to some row of the tile
-  const int klo_first = chunk > 0 ? ((pos0 + q0) / chunk) * chunk : 0;  // first key the tile's first row sees
-  const int j_lo = klo_first / TP_BN;
-  const int niter = (kv_end + TP_BN - 1) / TP_BN - j_lo;
+  // first key that a position sees (kept tokens aside)
+  auto first_key = [&](int pos) {
+    int k = chunk > 0 ? (pos / chunk) * chunk : 0;
+    if (window > 0 && pos - window + 1 > k) k = pos - window + 1;
+    return k;
+  };
+  const int j_lo = first_key(pos0 + q0) / TP_BN;
+  const int nkeep = min(j_lo, (keep + TP_BN - 1) / TP_BN);          // key steps of kept tokens before the window's
+  const int niter = nkeep + (kv_end + TP_BN - 1) / TP_BN - j_lo;
+  auto key_step = [&](int it) { return it < nkeep ? it : j_lo + it - nkeep; };
   const int nblk_seq = (pos0 + n_new + TP_BLK - 1) / TP_BLK;        // valid entries of bt_row
 
   extern __shared__ uint8_t smem_raw[];
@@ -191,7 +200,7 @@ __global__ void __launch_bounds__(TP_THREADS, 1)
         const int piece = is_k ? HALFK : TP_HALF, rowb = is_k ? KROW : 128;
         const int nm = (is_k && MAPS) ? 2 : 1;
         for (int it = 0; it < niter; ++it) {
-          const int s = it % TP_ST, j = j_lo + it;
+          const int s = it % TP_ST, j = key_step(it);
           if (it >= TP_ST) mbar_wait(&empty[s], (uint32_t)(it / TP_ST - 1) & 1u);
           mbar_expect_tx(&full[s], (uint32_t)tile);
           uint8_t* dst = ring + (size_t)s * tile;
@@ -297,8 +306,8 @@ __global__ void __launch_bounds__(TP_THREADS, 1)
       const uint32_t s_addr = lane_base + (uint32_t)t * 128u;  // S_t; the weights' hi terms over its first 64 columns, lo over the rest
       const uint32_t o_addr = lane_base + 256u + (uint32_t)t * 128u;
       const int qpos = pos0 + q0 + row;
-      const int klo = chunk > 0 ? (qpos / chunk) * chunk : 0;                             // first key this row sees
-      const int klo_last = chunk > 0 ? ((pos0 + q0 + TP_BM - 1) / chunk) * chunk : 0;     // ... and the tile's last row
+      const int klo = first_key(qpos);                          // first key this row sees
+      const int klo_last = first_key(pos0 + q0 + TP_BM - 1);    // ... and the tile's last row
       constexpr float LOG2E = 1.4426950408889634f;
       const float scale_log2 = scale * LOG2E;
       // capped scores, in log2 units: cap * log2e * tanh(s * scale / cap), tanh(x) = 1 - 2 / (1 + e^(2x))
@@ -309,7 +318,7 @@ __global__ void __launch_bounds__(TP_THREADS, 1)
       for (int it = 0; it < niter; ++it) {
         mbar_wait(&s_full[t], (uint32_t)it & 1u);
         tc_fence_after();
-        const int k0 = (j_lo + it) * TP_BN;
+        const int k0 = key_step(it) * TP_BN;
         const bool masked = k0 + TP_BN - 1 > pos0 + q0 || k0 < klo_last;  // some key of the step is hidden from some row
         uint32_t sv[TP_BN];
         auto load_scores = [&]() {
@@ -326,7 +335,7 @@ __global__ void __launch_bounds__(TP_THREADS, 1)
           if (masked) {
 #pragma unroll
             for (int i = 0; i < TP_BN; ++i)
-              if (k0 + i > qpos || k0 + i < klo) sv[i] = 0xff800000u;
+              if (k0 + i > qpos || (k0 + i < klo && k0 + i >= keep)) sv[i] = 0xff800000u;
           }
         };
         load_scores();
@@ -434,7 +443,7 @@ template <int DK, int DV, int KIND, bool MAPS>
 static int tp_launch(const CUtensorMap& km, const CUtensorMap& vm, const float* q, int ldq, const int32_t* block_table,
                      int64_t bt_stride, const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_pos0, int B,
                      int max_new, void* out, int H, int G, int chunk, float scale, float softcap, const float* sig_bias,
-                     int out_f32, int split_p, cudaStream_t stream) {
+                     int out_f32, int split_p, int window, int keep, cudaStream_t stream) {
   auto kern = swa_prefill_tc_kernel<DK, DV, KIND, MAPS>;
   // operand tiles + barriers + alignment slack; never less than half an SM's shared memory, so that one CTA (which takes all
   // 512 columns of tensor memory) is resident per SM
@@ -450,7 +459,7 @@ static int tp_launch(const CUtensorMap& km, const CUtensorMap& vm, const float* 
   const int gy = tpc >= 2 ? ((ny + tpc - 1) / tpc) * tpc : ny;  // the launch order of the kernel's tile map
   dim3 grid(MAPS ? (G / 2) * rep : G * ((rep + 1) / 2), gy, B);
   B200_CUDA_OK(launch_kernel(kern, grid, dim3(TP_THREADS), smem, stream, km, vm, q, ldq, block_table, bt_stride, seq_start,
-                             seq_slot, seq_pos0, out, H, G, chunk, scale, softcap, sig_bias, out_f32, split_p, ny));
+                             seq_slot, seq_pos0, out, H, G, chunk, scale, softcap, sig_bias, out_f32, split_p, ny, window, keep));
   return B200_OK;
 }
 
@@ -472,7 +481,9 @@ int b200_swa_sink_attn_prefill_tc(const float* q, int ldq, const void* k_pool, c
                                   const int32_t* block_table, int64_t bt_stride, const int32_t* seq_start,
                                   const int32_t* seq_slot, const int32_t* seq_pos0, int B, int max_new, float scale, void* out,
                                   int H, int G, int D, int Dv, int block_size, int chunk, float softcap,
-                                  const float* sigmoid_bias, int v_div, int out_f32, int split_p, void* stream) {
+                                  const float* sigmoid_bias, int v_div, int out_f32, int split_p, int window, int keep,
+                                  void* stream) {
+  B200_REQUIRE(window >= 0 && keep >= 0, "swa_sink_attn_prefill_tc: window %d, %d kept tokens", window, keep);
   B200_REQUIRE(q && k_pool && v_pool && block_table && seq_start && seq_slot && seq_pos0 && out,
                "swa_sink_attn_prefill_tc: null pointer");
   B200_REQUIRE(H > 0 && G > 0 && H % G == 0 && chunk >= 0 && v_div >= 1 && G % v_div == 0,
@@ -494,7 +505,7 @@ int b200_swa_sink_attn_prefill_tc(const float* q, int ldq, const void* k_pool, c
   cudaStream_t st = (cudaStream_t)stream;
 #define TP_GO(DK_, DV_, KIND_, MAPS_)                                                                                          \
   return tp_launch<DK_, DV_, KIND_, MAPS_>(km, vm, q, ldq, block_table, bt_stride, seq_start, seq_slot, seq_pos0, B, max_new, \
-                                           out, H, G, chunk, scale, softcap, sigmoid_bias, out_f32, split_p, st)
+                                           out, H, G, chunk, scale, softcap, sigmoid_bias, out_f32, split_p, window, keep, st)
   if (v_div == 2 && D == 32) {
     if (Dv == 64) TP_GO(32, 64, TP_SOFTMAX, true);
     TP_GO(32, 128, TP_SOFTMAX, true);

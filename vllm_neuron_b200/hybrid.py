@@ -59,6 +59,20 @@ The mixer 'parallel' is two mixers side by side over the same input, left_scale 
 Feed-forward: SiLU experts chosen by the largest softmax scores over all experts, weighed on their outputs by the chosen
 scores divided by their sum, times router.scale.
 
+A fifth block style, layer norm AFTER the sum (the "Goponex" design):
+  x <- LN(a x + mixer(x)),  x <- LN(a x + ff(x))   with LN a layer norm with a weight and no bias, a = postln_alpha; the
+sublayers read x itself.  Mixers:
+  * 'parallel' -- half the sum of two mixers over the same input, each RMS-normed over the width first:
+      left:  rotating attention (`RotAttnSpec`) whose values are the keys as projected, per-head RMS norms on q and k,
+             neighbour-pair rotation with YaRN blending, a sliding window beside which the first mask.keep_first tokens stay
+             visible;
+      right: a selective state-space scan with a step size per channel (`MambaSpec`): in-projection -> [x | z], short convolution
+             + SiLU on x, x-projection -> [dt rank | B | C], S <- exp(dt A) S + dt x B^T, y = S C + D x, y silu(z), out-projection.
+             State per sequence: S (fp32) and the last taps - 1 convolution inputs;
+  * 'mlstm'    -- matrix memory with exponential input gates under a running maximum and a normaliser (`MatrixMemorySpec`), a
+             per-head RMS norm, a sigmoid output gate.  State per sequence: S, the normaliser and the maximum (fp32).
+Feed-forward: W_down relu(W_up h)^2 with biases, or none.
+
 The step is ONE ragged batch (`StepMeta`): portions of prompts and single decoded tokens run through the same kernels, each
 sequence continuing from its KV pages (block table row) and its state slot.  fp32 everywhere the design asks for it
 (residual stream, norms, softmax, router, recurrence); GEMM operands, weights and KV pools are bf16, or fp32 when the model is
@@ -78,7 +92,8 @@ from . import ops
 
 ARCHITECTURE = "Pumopel"
 # block style per architecture: how the norms sit around the sublayers (and which norm it is)
-BLOCK_STYLES = {"Pumopel": "dyt_sandwich", "Kenetar": "rms_post", "Zudarax": "rms_parallel", "Gerupel": "rms_dual"}
+BLOCK_STYLES = {"Pumopel": "dyt_sandwich", "Kenetar": "rms_post", "Zudarax": "rms_parallel", "Gerupel": "rms_dual",
+                "Goponex": "ln_post"}
 ROT_ATTN_KINDS = ("attention", "attention_2", "attention_3")  # the parallel style's mixers
 _NO_WINDOW = 1 << 30
 
@@ -202,6 +217,9 @@ class RotAttnSpec:
     pool: int = 0            # > 0 (with a window): blocks of this many positions wholly before the window are one key / value each
     unit_sink: bool = False  # softmax with 1 added to its denominator
     temp: bool = False       # a per-head factor on the scores
+    head_norm: bool = False  # RMS norm of every q and k head, weights per column of a head
+    v_from_k: bool = False   # the values are the keys as projected, before norm and rotation (no value projection)
+    keep: int = 0            # > 0 (with a window): the sequence's first `keep` tokens stay visible
 
     @property
     def maps(self) -> int:
@@ -233,12 +251,38 @@ class GatedScanSpec:
 
 
 @dataclass
+class MambaSpec:
+    """Selective scan with a step size per channel: `inner` channels of `state` states each, step sizes through a bottleneck of
+    `dt_rank` columns, a short convolution of `conv` taps."""
+    inner: int
+    state: int
+    dt_rank: int
+    conv: int
+
+    @property
+    def rank_cols(self) -> int:  # columns the step-size bottleneck takes in its GEMM operand (zero-padded to whole 16-byte pieces)
+        return -(-self.dt_rank // 8) * 8
+
+
+@dataclass
+class MatrixMemorySpec:
+    """Matrix memory with exponential gates per head: q, k have `dim` columns, v has `vdim`; raw gates pass through
+    gate_cap * tanh(. / gate_cap)."""
+    heads: int
+    dim: int
+    vdim: int
+    gate_cap: float
+
+
+@dataclass
 class DualMixerSpec:
-    """Two mixers side by side over the same input: left_scale * attention + right_scale * recurrence."""
+    """Two mixers side by side over the same input: left_scale * attention + right_scale * recurrence.  branch_norm: each output is
+    RMS-normed over the model width before it is scaled."""
     left: RotAttnSpec
-    right: GatedScanSpec
+    right: GatedScanSpec | MambaSpec
     left_scale: float
     right_scale: float
+    branch_norm: bool = False
 
 
 @dataclass
@@ -265,6 +309,7 @@ class MoeSpec:
 @dataclass
 class DenseSpec:
     ff: int
+    act: str = "gelu_glu"  # 'gelu_glu': down(gelu_tanh(gate h) * up h); 'relu2': down(relu(up h)^2), projections with biases
 
 
 @dataclass
@@ -287,6 +332,7 @@ class HybridConfig:
     norm_groups: int = 1         # parallel style: equal parts of a row that are normed on their own
     residual_mult: float = 1.0   # dual-norm style: factor on the sum of a layer's branches
     loop: dict | None = None     # dual-norm style: start, stop, times -- layers [start, stop) run `times` times in a row
+    postln_alpha: float = 1.0    # layer-norm-after-the-sum style: factor on x in the sum
 
     @property
     def style(self) -> str:
@@ -309,9 +355,12 @@ class HybridConfig:
         post = BLOCK_STYLES[name] == "rms_post"
         par = BLOCK_STYLES[name] == "rms_parallel"
         dual = BLOCK_STYLES[name] == "rms_dual"
+        lnp = BLOCK_STYLES[name] == "ln_post"
         for L in d["layers"]:
             m = L["mixer"]
-            if dual:
+            if lnp:
+                mixer = _post_ln_mixer(L["type"], m, name)
+            elif dual:
                 if L["type"] != "parallel":
                     raise ValueError(f"layer type {L['type']!r} is not part of the {name} design")
                 r = m["right"]
@@ -345,13 +394,17 @@ class HybridConfig:
                     raise ValueError(f"latent attention: {mixer.rot.dims} rotating columns in a rotated part of {mixer.rot_dim}")
             else:
                 raise ValueError(f"unknown layer type {L['type']!r}")
-            if not par and not dual and post != (L["type"] in ("delta", "latent_attention")):
+            if not par and not dual and not lnp and post != (L["type"] in ("delta", "latent_attention")):
                 raise ValueError(f"layer type {L['type']!r} is not part of the {name} design")
             f = L.get("mlp")
             mlp = None
             if f:
                 kind = f.get("kind", "moe")
-                if dual:
+                if lnp:
+                    if kind != "dense":
+                        raise ValueError(f"unknown feed-forward kind {kind!r}")
+                    mlp = DenseSpec(int(f["ff"]), "relu2")
+                elif dual:
                     if kind != "moe":
                         raise ValueError(f"unknown feed-forward kind {kind!r}")
                     mlp = MoeSpec(int(f["router"]["experts"]), int(f["router"]["top"]), int(f["expert"]["ff"]), route="softmax_renorm",
@@ -385,7 +438,8 @@ class HybridConfig:
                 raise ValueError(f"loop {loop} over {len(layers)} layers")
         return HybridConfig(int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), float(emb.get("scale", 1.0)), layers, name,
                             {k: int(big[k]) for k in ("buckets", "mul_prev", "mul_cur")} if big else None,
-                            float(d.get("logit_scale", 1.0)), groups, float(d.get("residual_mult", 1.0)) if dual else 1.0, loop)
+                            float(d.get("logit_scale", 1.0)), groups, float(d.get("residual_mult", 1.0)) if dual else 1.0, loop,
+                            float(d["postln_alpha"]) if lnp else 1.0)
 
     @staticmethod
     def from_pretrained(path: str) -> "HybridConfig":
@@ -408,6 +462,9 @@ class HybridConfig:
             out["residual_mult"] = self.residual_mult
             if self.loop:
                 out["loop"] = dict(self.loop)
+        if self.style == "ln_post":
+            del out["embedding"]
+            out["postln_alpha"] = self.postln_alpha
         for L in self.layers:
             m = L.mixer
             if isinstance(m, DualMixerSpec):
@@ -418,9 +475,14 @@ class HybridConfig:
                     if a.rot.scaling:
                         left["rot"]["scaling"] = dict(a.rot.scaling)
                 if a.window:
-                    left["mask"] = {"size": a.window, **({"pool": a.pool} if a.pool else {})}
-                mixer = {"left": left, "right": {"heads": r.heads, "dim": r.dim, "vdim": r.vdim}, "left_scale": m.left_scale,
-                         "right_scale": m.right_scale}
+                    left["mask"] = {"size": a.window, **({"pool": a.pool} if a.pool else {}), **({"keep_first": a.keep} if a.keep else {})}
+                if isinstance(r, MambaSpec):
+                    mixer = {"left": left, "right": {"inner": r.inner, "state": r.state, "dt_rank": r.dt_rank, "conv": r.conv}}
+                else:
+                    mixer = {"left": left, "right": {"heads": r.heads, "dim": r.dim, "vdim": r.vdim}, "left_scale": m.left_scale,
+                             "right_scale": m.right_scale}
+            elif isinstance(m, MatrixMemorySpec):
+                mixer = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "gate_cap": m.gate_cap}
             elif isinstance(m, RotAttnSpec):
                 mixer = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
                          "rot": {"dims": m.rot.dims, "base": m.rot.base}}
@@ -505,6 +567,37 @@ def _window_pool_attn_spec(m: dict) -> RotAttnSpec:
     return spec
 
 
+def _post_ln_mixer(kind: str, m: dict, name: str):
+    """One of the layer-norm-after-the-sum style's mixers from its configuration entry."""
+    if kind == "mlstm":
+        mm = MatrixMemorySpec(int(m["heads"]), int(m["dim"]), int(m["vdim"]), float(m["gate_cap"]))
+        if mm.gate_cap <= 0:
+            raise ValueError(f"mlstm layer: gate_cap {mm.gate_cap}")
+        return mm
+    if kind != "parallel":
+        raise ValueError(f"layer type {kind!r} is not part of the {name} design")
+    a, r = m["left"], m["right"]
+    rot = a.get("rot")
+    rot = RotSpec(int(rot["dims"]), float(rot["base"]), dict(rot["scaling"]) if rot.get("scaling") else None) if rot else None
+    left = RotAttnSpec(int(a["heads"]), int(a["kv_heads"]), int(a["dim"]), int(a["vdim"]), float(a["scale"]), rot, head_norm=True,
+                       v_from_k=True)
+    if left.heads % left.kv_heads:
+        raise ValueError(f"parallel layer: {left.heads} query heads over {left.kv_heads} kv heads")
+    if left.vdim != left.dim:
+        raise ValueError(f"parallel layer: the values are the keys, so vdim {left.vdim} must equal dim {left.dim}")
+    if rot is not None and (rot.dims % 2 or rot.dims > left.dim):
+        raise ValueError(f"parallel layer: {rot.dims} rotating columns in heads of {left.dim}")
+    mask = a.get("mask") or {}
+    left.window = int(mask.get("size") or 0)
+    left.keep = int(mask.get("keep_first") or 0) if left.window else 0
+    if left.window < 0 or left.keep < 0:
+        raise ValueError(f"parallel layer: window {left.window}, {left.keep} kept tokens")
+    right = MambaSpec(int(r["inner"]), int(r["state"]), int(r["dt_rank"]), int(r["conv"]))
+    if min(right.inner, right.state, right.dt_rank, right.conv) < 1:
+        raise ValueError(f"parallel layer: {right}")
+    return DualMixerSpec(left, right, 0.5, 0.5, branch_norm=True)
+
+
 def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple]:
     """Checkpoint tensor name -> shape (a linear layer's matrix has one row per output)."""
     W = cfg.width
@@ -521,8 +614,10 @@ def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple]:
         if cfg.loop:
             s["loop.step"] = (cfg.loop["times"], W)
 
+    lnp = cfg.style == "ln_post"
+
     def norm(n):
-        if post or par or dual:
+        if post or par or dual or lnp:
             s[n] = (W,)
         else:
             s[n], s[n + ".b"], s[n + ".alpha"] = (W,), (W,), ()
@@ -530,11 +625,23 @@ def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple]:
     norm("final.norm")
     for i, L in enumerate(cfg.layers):
         p = f"l{i}."
-        for n in ("norm1",) if par else (("norm1",) + (("norm2",) if L.mlp else ())) if post or dual else \
+        for n in ("norm1",) if par else (("norm1",) + (("norm2",) if L.mlp else ())) if post or dual or lnp else \
                 (("norm1", "norm1b") + (("norm2", "norm2b") if L.mlp else ())):
             norm(p + n)
         m = L.mixer
-        if isinstance(m, DualMixerSpec):
+        if isinstance(m, DualMixerSpec) and isinstance(m.right, MambaSpec):
+            a, r = m.left, m.right
+            s.update({p + "mix.left.q": (a.q_cols, W), p + "mix.left.k": (a.k_cols, W), p + "mix.left.q.norm": (a.dim,),
+                      p + "mix.left.k.norm": (a.dim,), p + "mix.left.o": (W, a.heads * a.vdim), p + "mix.left.out": (W,),
+                      p + "mix.right.in": (2 * r.inner, W), p + "mix.right.conv": (r.inner, r.conv), p + "mix.right.conv.b": (r.inner,),
+                      p + "mix.right.x": (r.dt_rank + 2 * r.state, r.inner), p + "mix.right.dt": (r.inner, r.dt_rank),
+                      p + "mix.right.dt.b": (r.inner,), p + "mix.right.A_log": (r.inner, r.state), p + "mix.right.D": (r.inner,),
+                      p + "mix.right.o": (W, r.inner), p + "mix.right.out": (W,)})
+        elif isinstance(m, MatrixMemorySpec):
+            s.update({p + "mix.q": (m.heads * m.dim, W), p + "mix.k": (m.heads * m.dim, W), p + "mix.v": (m.heads * m.vdim, W),
+                      p + "mix.g": (m.heads * m.vdim, W), p + "mix.o": (W, m.heads * m.vdim), p + "mix.norm": (m.heads * m.vdim,),
+                      p + "mix.i": (m.heads, W), p + "mix.i.b": (m.heads,), p + "mix.f": (m.heads, W), p + "mix.f.b": (m.heads,)})
+        elif isinstance(m, DualMixerSpec):
             a, r = m.left, m.right
             s.update({p + "mix.left.q": (a.q_cols, W), p + "mix.left.k": (a.k_cols, W), p + "mix.left.v": (a.v_cols, W),
                       p + "mix.left.temp": (a.heads,), p + "mix.left.o": (W, a.heads * a.vdim),
@@ -581,6 +688,8 @@ def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple]:
         f = L.mlp
         if isinstance(f, PolySpec):
             s.update({p + "mlp.up": (f.ff, W), p + "mlp.down": (W, f.ff), p + "mlp.act": (4,)})
+        elif isinstance(f, DenseSpec) and f.act == "relu2":
+            s.update({p + "mlp.up": (f.ff, W), p + "mlp.up.b": (f.ff,), p + "mlp.down": (W, f.ff), p + "mlp.down.b": (W,)})
         elif isinstance(f, DenseSpec):
             s.update({p + "mlp.gate": (f.ff, W), p + "mlp.up": (f.ff, W), p + "mlp.down": (W, f.ff)})
         elif f:
@@ -614,6 +723,10 @@ def random_weights(cfg: HybridConfig, seed: int = 0, std: float | None = None) -
             t = 0.9 * torch.rand(shape, generator=g)
         elif leaf == "step":
             t = 0.2 * torch.randn(shape, generator=g)
+        elif cfg.style == "ln_post" and name.endswith(".dt.b"):
+            t = -4.0 + 2.5 * torch.rand(shape, generator=g)  # small steps: the scan remembers
+        elif cfg.style == "ln_post" and name.endswith("mix.f.b"):
+            t = 2.0 + 3.0 * torch.rand(shape, generator=g)  # forget gates near one
         elif leaf == "b" and len(shape) == 1:
             t = 0.05 * torch.randn(shape, generator=g)
         elif leaf == "act":
@@ -622,7 +735,7 @@ def random_weights(cfg: HybridConfig, seed: int = 0, std: float | None = None) -
             t = -2.0 + torch.randn(shape, generator=g)
         elif leaf in ("lq1", "lk1", "lq2", "lk2"):
             t = 0.3 * torch.randn(shape, generator=g)
-        elif leaf in ("norm1", "norm2", "norm1b", "norm2b", "norm") and len(shape) == 1:
+        elif leaf in ("norm1", "norm2", "norm1b", "norm2b", "norm", "out") and len(shape) == 1:
             t = 1.0 + 0.1 * torch.randn(shape, generator=g)
         elif leaf == "A_log":
             t = torch.log(0.5 + 1.5 * torch.rand(shape, generator=g))
@@ -753,9 +866,10 @@ class HybridCausalLM:
         post = cfg.style == "rms_post"
         par = cfg.style == "rms_parallel"
         dual = cfg.style == "rms_dual"
+        lnp = cfg.style == "ln_post"
 
         def norm(name):
-            if post or par or dual:  # RMS norm: weight stored around zero (post-norm) or plain (in groups: parallel)
+            if post or par or dual or lnp:  # weight stored around zero (post-norm) or plain (RMS in groups: parallel; layer norm)
                 return vec(name)
             return (vec(name), vec(name + ".b"), float(get(name + ".alpha").float()))
 
@@ -778,9 +892,40 @@ class HybridCausalLM:
         for i, L in enumerate(cfg.layers):
             p, m = f"l{i}.", L.mixer
             lw = {"spec": L, "norm1": norm(p + "norm1")}
-            if not post and not par and not dual:
+            if not post and not par and not dual and not lnp:
                 lw["norm1b"] = norm(p + "norm1b")
-            if isinstance(m, DualMixerSpec):
+            if isinstance(m, DualMixerSpec) and isinstance(m.right, MambaSpec):
+                a, r = m.left, m.right
+                if a.rot is not None:
+                    key = (a.rot.dims, a.rot.base, json.dumps(a.rot.scaling, sort_keys=True))
+                    if key not in rot_tables:
+                        rot_tables[key] = tuple(t.to(dev) for t in a.rot.tables(self.max_blocks * block_size))
+                    lw["rot"] = rot_tables[key]
+                # the step-size bottleneck's columns are padded with zeros to whole 16-byte pieces (its second GEMM's operand rows)
+                pad = r.rank_cols - r.dt_rank
+                wx, wdt = get(p + "mix.right.x"), get(p + "mix.right.dt")
+                wx = torch.cat([wx[:r.dt_rank], wx.new_zeros((pad, r.inner)), wx[r.dt_rank:]])
+                wdt = torch.cat([wdt, wdt.new_zeros((r.inner, pad))], dim=1)
+                lw.update(  # ONE GEMM for everything that reads x: [left q | k | right x | z]
+                    w_in=lin(p + "mix.left.q", p + "mix.left.k", p + "mix.right.in"), w_o=lin(p + "mix.left.o"), w_o2=lin(p + "mix.right.o"),
+                    q_norm=vec(p + "mix.left.q.norm"), k_norm=vec(p + "mix.left.k.norm"), out1=vec(p + "mix.left.out"),
+                    out2=vec(p + "mix.right.out"), conv_w=vec(p + "mix.right.conv"), conv_b=vec(p + "mix.right.conv.b"),
+                    w_x=wx.to(dev, et).contiguous(), w_dt=wdt.to(dev, et).contiguous(), dt_b=vec(p + "mix.right.dt.b"),
+                    a_log2=(-torch.exp(get(p + "mix.right.A_log").double()) * math.log2(math.e)).to(dev, torch.float32).contiguous(),
+                    d=vec(p + "mix.right.D"),
+                    k_pool=torch.zeros((num_blocks, a.kv_heads, block_size, a.dim), dtype=et, device=dev),
+                    v_pool=torch.zeros((num_blocks, a.kv_heads, block_size, a.vdim), dtype=et, device=dev),
+                    conv_state=torch.zeros((slots, max(r.conv - 1, 1), r.inner), dtype=torch.float32, device=dev),
+                    scan_state=torch.zeros((slots, r.inner, r.state), dtype=torch.float32, device=dev))
+            elif isinstance(m, MatrixMemorySpec):
+                # gate rows last and the row count padded to whole 16-byte pieces of fp32: q, k, v and g stay on the 16-byte grid
+                w_in = torch.cat([get(p + "mix." + n) for n in "qkvgif"])
+                w_in = torch.cat([w_in, w_in.new_zeros((-w_in.shape[0] % 4, cfg.width))])
+                lw.update(w_in=w_in.to(dev, et).contiguous(), w_o=lin(p + "mix.o"), onorm=vec(p + "mix.norm"), i_bias=vec(p + "mix.i.b"),
+                          f_bias=vec(p + "mix.f.b"),
+                          scan_state=torch.zeros((slots, m.heads, m.vdim + 1, m.dim), dtype=torch.float32, device=dev),
+                          max_state=torch.zeros((slots, m.heads), dtype=torch.float32, device=dev))
+            elif isinstance(m, DualMixerSpec):
                 a, r = m.left, m.right
                 if a.rot is not None:
                     key = (a.rot.dims, a.rot.base, json.dumps(a.rot.scaling, sort_keys=True))
@@ -861,10 +1006,12 @@ class HybridCausalLM:
             f = L.mlp
             if f and not par:
                 lw["norm2"] = norm(p + "norm2")
-                if not post and not dual:
+                if not post and not dual and not lnp:
                     lw["norm2b"] = norm(p + "norm2b")
             if isinstance(f, PolySpec):  # W_up rides in w_in
                 lw.update(w_down=lin(p + "mlp.down"), act=vec(p + "mlp.act"))
+            elif isinstance(f, DenseSpec) and f.act == "relu2":
+                lw.update(w_up=lin(p + "mlp.up"), up_b=vec(p + "mlp.up.b"), w_down=lin(p + "mlp.down"), down_b=vec(p + "mlp.down.b"))
             elif isinstance(f, DenseSpec):
                 lw.update(w_gu=lin(p + "mlp.gate", p + "mlp.up"), w_down=lin(p + "mlp.down"))
             elif f:
@@ -904,6 +1051,9 @@ class HybridCausalLM:
         es = 2 if self.et == torch.bfloat16 else 4
         if self.cfg.style == "rms_dual":  # per run: K / V rows of a page and its pooled-block rows
             return sum(sum(t.shape[1] * t.shape[2] * t.shape[3] * es for n, t in run.items() if n.endswith("_pool")) for run in self.runs)
+        if self.cfg.style == "ln_post":
+            return sum(L.mixer.left.kv_heads * self.block_size * (L.mixer.left.dim + L.mixer.left.vdim) * es
+                       for L in self.cfg.layers if isinstance(L.mixer, DualMixerSpec))
         return sum(L.mixer.kv_heads * self.block_size * (L.mixer.dim * getattr(L.mixer, "maps", 1) + L.mixer.vdim) * es
                    for L in self.cfg.layers if isinstance(L.mixer, (AttnSpec, RotAttnSpec))) + \
             sum(self.block_size * (L.mixer.kv_rank + L.mixer.rot_dim) * es for L in self.cfg.layers if L.kind == "latent_attention")
@@ -911,6 +1061,8 @@ class HybridCausalLM:
     def state_bytes_per_slot(self) -> int:
         if self.cfg.style == "rms_dual":
             return sum(4 * run["scan_state"][0].numel() for run in self.runs)
+        if self.cfg.style == "ln_post":
+            return sum(4 * lw[n][0].numel() for lw in self.layers for n in ("scan_state", "conv_state", "max_state") if n in lw)
         return sum(4 * (L.mixer.heads * L.mixer.state * L.mixer.vdim + (L.mixer.conv - 1) * L.mixer.channels)
                    for L in self.cfg.layers if L.kind == "mamba2") + \
             sum(4 * (L.mixer.heads * L.mixer.dim * L.mixer.vdim + (L.mixer.conv - 1) * L.mixer.channels)
@@ -1088,6 +1240,64 @@ class HybridCausalLM:
         self.last_logits = self._linear(h1.index_select(0, logit_rows).contiguous(), self.head)
         return self.last_logits
 
+    def _keep_mamba_mixer(self, lw, h, meta):
+        """Both halves of the layer-norm style's 'parallel' mixer -> (attention branch, state-space branch), fp32 [T, W] each, before
+        their norms."""
+        m = lw["spec"].mixer
+        a, r, et = m.left, m.right, self.et
+        proj = self._linear(h, lw["w_in"])  # fp32 [T, left q | k | right x | z]
+        k0, x0 = a.q_cols, a.q_cols + a.k_cols
+        z0 = x0 + r.inner
+        cos, sin = lw.get("rot", (None, None))
+        q = ops.qk_norm_rope_kv_write(proj, 0, k0, k0, a.heads, lw["k_pool"], lw["v_pool"], meta, q_norm=lw["q_norm"], k_norm=lw["k_norm"],
+                                      eps=self.cfg.eps, rot_n=a.rot.dims if a.rot else 0, rot_half=False, cos=cos, sin=sin, head_norm=True)
+        att = ops.swa_sink_attn(q, a.heads, lw["k_pool"], lw["v_pool"], self.block_table, meta, None, a.scale, a.window or _NO_WINDOW,
+                                split_p=True, keep=a.keep)
+        x = ops.causal_conv_silu(proj, x0, r.inner, lw["conv_w"], lw["conv_b"], lw["conv_state"], meta, et)
+        xp = self._linear(x, lw["w_x"])  # fp32 [T, dt bottleneck | B | C]
+        low = xp[:, :r.rank_cols] if et == torch.float32 else ops.bias_act(xp, 0, r.rank_cols, None, ops.ACT_NONE, et)
+        dt = self._linear(low, lw["w_dt"])
+        y = ops.selective_scan(x, dt, xp, r.rank_cols, r.rank_cols + r.state, proj[:, z0:], lw["a_log2"], lw["dt_b"], lw["d"],
+                               lw["scan_state"], meta)
+        return self._linear(att, lw["w_o"]), self._linear(y, lw["w_o2"])
+
+    def _mlstm(self, lw, h, meta):
+        m = lw["spec"].mixer
+        proj = self._linear(h, lw["w_in"])  # fp32 [T, q | k | v | g | i | f]
+        k0, v0 = m.heads * m.dim, 2 * m.heads * m.dim
+        g0 = v0 + m.heads * m.vdim
+        i0 = g0 + m.heads * m.vdim
+        o, nq, floor = ops.matrix_memory(proj, 0, k0, v0, i0, i0 + m.heads, lw["i_bias"], lw["f_bias"], m.gate_cap, lw["scan_state"],
+                                         lw["max_state"], meta, m.heads, m.dim, m.vdim)
+        u = ops.matrix_memory_out(o, nq, floor, m.dim ** -0.5, proj, g0, lw["onorm"], self.cfg.eps, m.heads, self.et)
+        return self._linear(u, lw["w_o"])
+
+    def _forward_post_ln(self, tokens, meta, logit_rows, capture):
+        """x <- LN(a x + mixer(x)); x <- LN(a x + ff(x)): one pass over the residual per sublayer norms the branches, adds, norms the sum
+        and writes the next GEMM's operand."""
+        et, cfg = self.et, self.cfg
+        alpha, eps = cfg.postln_alpha, cfg.eps
+        x, h = ops.embed_bigram(tokens, self.embed, 1.0, meta)
+        for lw in self.layers:
+            m = lw["spec"].mixer
+            if isinstance(m, DualMixerSpec):
+                y1, y2 = self._keep_mamba_mixer(lw, h, meta)
+                h = ops.postln_residual(x, alpha, lw["norm1"], eps, y1=y1, w1=lw["out1"], y2=y2, w2=lw["out2"], c=m.left_scale, out_dtype=et)
+            else:
+                h = ops.postln_residual(x, alpha, lw["norm1"], eps, y1=self._mlstm(lw, h, meta), out_dtype=et)
+            f = lw["spec"].mlp
+            if f:
+                u = ops.bias_act(self._linear(h, lw["w_up"]), 0, f.ff, lw["up_b"], ops.ACT_RELU2, et)
+                h = ops.postln_residual(x, alpha, lw["norm2"], eps, y1=self._linear(u, lw["w_down"]), vec=lw["down_b"], out_dtype=et)
+            if capture is not None:
+                capture.append(x.clone())
+        if logit_rows is None or logit_rows.numel() == 0:
+            self.last_logits = None
+            return None
+        hf = ops.postln_residual(x.index_select(0, logit_rows).contiguous(), 1.0, self.final_norm, eps, out_dtype=et, store=False)
+        self.last_logits = self._linear(hf, self.head)
+        return self.last_logits
+
     def _post_ff(self, lw, h):
         """Feed-forward of the post-norm style -> (fp32 branch rows, rows per token, their weights or None)."""
         f = lw["spec"].mlp
@@ -1139,6 +1349,8 @@ class HybridCausalLM:
             return self._forward_post(tokens, meta, logit_rows, capture)
         if self.cfg.style == "rms_parallel":
             return self._forward_parallel(tokens, meta, logit_rows, capture)
+        if self.cfg.style == "ln_post":
+            return self._forward_post_ln(tokens, meta, logit_rows, capture)
         if self.cfg.style == "rms_dual":
             return self._forward_dual(tokens, meta, logit_rows, capture)
         et, n = self.et, len(self.layers)

@@ -10,7 +10,8 @@ import os
 import torch
 
 from . import _cabi
-from ._cabi import ACT_GELU_TANH, ACT_SILU, ACT_SWISH_CLAMPED, BF16, F32, FP8_E4M3, INT8, ROUTE_SIGMOID, ROUTE_SOFTMAX_RENORM, ROUTE_SOFTMAX_TOP, check
+from ._cabi import (ACT_GELU_TANH, ACT_NONE, ACT_RELU2, ACT_SILU, ACT_SWISH_CLAMPED, BF16, F32, FP8_E4M3, INT8, ROUTE_SIGMOID,
+                    ROUTE_SOFTMAX_RENORM, ROUTE_SOFTMAX_TOP, check)
 
 _QDT = {None: BF16, "bf16": BF16, "fp8": FP8_E4M3, "int8": INT8}
 _TORCH_Q = {FP8_E4M3: torch.float8_e4m3fn, INT8: torch.int8}
@@ -738,7 +739,7 @@ _SWA_PREFILL_LEGACY = bool(os.environ.get("B200_SWA_PREFILL_LEGACY"))
 
 def swa_sink_attn(q_src, num_heads: int, k_pool, v_pool, block_table, meta, sink, scale: float, window: int,
                   latent_values: int = 0, *, chunk: int = 0, softcap: float = 0.0, sigmoid_bias=None, out_f32: bool = False,
-                  split_p: bool = False, pooled=None):
+                  split_p: bool = False, pooled=None, keep: int = 0):
     """q = the first num_heads * D columns of the fp32 rows q_src -> [T, num_heads * Dv] in the pools' element type.
     sink None: ordinary softmax.  latent_values = C > 0: v_pool is ignored and the values are the first C columns of the key
     rows (attention over cached latents: one pool holds both).
@@ -747,7 +748,11 @@ def swa_sink_attn(q_src, num_heads: int, k_pool, v_pool, block_table, meta, sink
     over keys.  A value pool with fewer heads than the key pool: consecutive key heads share a value head (two score maps over
     the same values).  out_f32: fp32 rows.  split_p: the tensor-core kernel carries the weights as two bf16 terms.
     pooled = (pooled key pool, pooled value pool, P) with a window: every block of P positions that lies wholly before a query's
-    window is seen as one key / value, the block's row of the pooled pools (kv_pool_mean), in the same softmax."""
+    window is seen as one key / value, the block's row of the pooled pools (kv_pool_mean), in the same softmax.
+    keep > 0 with a window: the sequence's first `keep` tokens stay visible to every later query."""
+    assert not (keep and (pooled is not None or latent_values))
+    if window >= (1 << 30):
+        keep = 0
     _cuda(q_src, k_pool, v_pool, block_table, sink, sigmoid_bias)
     pk, pv, pool = pooled if pooled is not None else (None, None, 0)
     if pool:
@@ -756,7 +761,7 @@ def swa_sink_attn(q_src, num_heads: int, k_pool, v_pool, block_table, meta, sink
         assert not latent_values and window < (1 << 30) and pk.dtype == k_pool.dtype and pv.dtype == k_pool.dtype
         assert pk.is_contiguous() and pv.is_contiguous() and pk.shape == (k_pool.shape[0], k_pool.shape[1], ppb, k_pool.shape[3])
         assert pv.shape == (v_pool.shape[0], v_pool.shape[1], ppb, v_pool.shape[3])
-    pool_args = (_ptr(pk), _ptr(pv), int(pool))
+    pool_args = (_ptr(pk), _ptr(pv), int(pool), int(keep))
     _f32(q_src, sink, sigmoid_bias)
     assert block_table.dtype == torch.int32 and block_table.stride(1) == 1
     _, g, bs, d = k_pool.shape
@@ -772,11 +777,11 @@ def swa_sink_attn(q_src, num_heads: int, k_pool, v_pool, block_table, meta, sink
     variant = (int(chunk), float(softcap), _ptr(sigmoid_bias), v_div, 1 if out_f32 else 0)
     plain = not chunk and not softcap and sigmoid_bias is None and v_div == 1 and not out_f32
     # the per-launch timer tells the variants apart (their floors differ)
-    tag = "" if plain and not pool else "[" + "+".join(n for n, on in (("chunk", chunk), ("cap", softcap), ("sigmoid", sigmoid_bias is not None),
-                                                                       ("maps", v_div > 1), ("pool", pool)) if on) + "]"
-    # long prompt portions in bf16 serving, head sizes of 64 / 128 with pages of 32 tokens: the tcgen05 kernel (128-row query
+    tag = "" if plain and not pool and not keep else "[" + "+".join(n for n, on in (("chunk", chunk), ("cap", softcap), ("sigmoid", sigmoid_bias is not None),
+                                                                       ("maps", v_div > 1), ("pool", pool), ("keep", keep)) if on) + "]"
+    # long prompt portions in bf16 serving (a sliding window only without pooled blocks), head sizes of 64 / 128 with pages of 32 tokens: the tcgen05 kernel (128-row query
     # tiles, accumulators in tensor memory); B200_SWA_PREFILL_LEGACY=1 keeps the mma.sync kernel (A/B aid)
-    if (k_pool.dtype == torch.bfloat16 and meta.max_new >= PREFILL_TC_MIN_TOKENS and sink is None and window >= (1 << 30)
+    if (k_pool.dtype == torch.bfloat16 and meta.max_new >= PREFILL_TC_MIN_TOKENS and sink is None and not pool
             and not latent_values and q_src.stride(0) % 4 == 0 and q_src.data_ptr() % 16 == 0 and not _SWA_PREFILL_LEGACY
             and _cabi.load().b200_swa_sink_attn_prefill_tc_supported(d, dv, bs, v_div, 1 if softcap else 0,
                                                                      0 if sigmoid_bias is None else 1)):
@@ -785,7 +790,8 @@ def swa_sink_attn(q_src, num_heads: int, k_pool, v_pool, block_table, meta, sink
                                                              _ptr(block_table), block_table.stride(0), _ptr(meta.seq_start),
                                                              _ptr(meta.seq_slot), _ptr(meta.seq_pos0), meta.num_seqs, meta.max_new,
                                                              float(scale), _ptr(out), num_heads, g, d, dv, bs, *variant,
-                                                             1 if split_p else 0, _stream()),
+                                                             1 if split_p else 0, int(window) if window < (1 << 30) else 0,
+                                                             int(keep), _stream()),
                   "b200_swa_sink_attn_prefill_tc")
         return out
     # shorter prompt portions in bf16 serving: the mma.sync kernel; decode-sized steps, fp32 pools and odd head sizes: one CTA
@@ -812,6 +818,7 @@ def swa_sink_attn(q_src, num_heads: int, k_pool, v_pool, block_table, meta, sink
     span = min(getattr(meta, "max_end", 0) or 0, int(window), int(chunk) if chunk else 1 << 30)
     if pool:  # the blocks before the window count as keys too
         span += max((getattr(meta, "max_end", 0) or 0) - int(window), 0) // pool
+    span += int(keep)
     tc = (k_pool.dtype == torch.bfloat16 and not latent_values and d % 16 == 0 and dv % 16 == 0 and d * v_div <= 512 and dv <= 256
           and q_src.stride(0) % 2 == 0)
     gv = g // v_div
@@ -1119,11 +1126,14 @@ def diff_head_norm_gate(a, lam: float, post: float, gate_src, gate_col0: int, ep
 
 
 def qk_norm_rope_kv_write(src, q_col0: int, k_col0: int, v_col0: int, heads: int, k_pool, v_pool, meta, *, q_norm=None,
-                          k_norm=None, eps: float = 0.0, rot_n: int = 0, rot_half: bool = True, cos=None, sin=None, q_head_scale=None):
+                          k_norm=None, eps: float = 0.0, rot_n: int = 0, rot_half: bool = True, cos=None, sin=None, q_head_scale=None,
+                          head_norm: bool = False):
     """fp32 rows src = [.. q: heads * D .. k: G * D .. v: Gv * Dv ..] -> q fp32 [T, heads * D] (normed over the whole projection
     when q_norm is given, leading rot_n columns of every head rotated by the token's position), and the step's keys (same
     treatment) and values written into the pools [num_blocks, G, block_size, D] / [num_blocks, Gv, block_size, Dv].
-    q_head_scale fp32 [heads]: q of head h is multiplied by it (a per-head temperature of the scores)."""
+    q_head_scale fp32 [heads]: q of head h is multiplied by it (a per-head temperature of the scores).
+    head_norm: the norms are per head, q_norm / k_norm fp32 [D] shared by the heads.  v_col0 may equal k_col0: the cached values
+    are then the keys as projected, before norm and rotation."""
     _cuda(src, k_pool, v_pool, q_norm, k_norm, cos, sin, q_head_scale)
     _f32(q_norm, k_norm, cos, sin, q_head_scale)
     assert q_head_scale is None or q_head_scale.numel() == heads
@@ -1132,6 +1142,8 @@ def qk_norm_rope_kv_write(src, q_col0: int, k_col0: int, v_col0: int, heads: int
     _, g, bs, d = k_pool.shape
     _, gv, _, dv = v_pool.shape
     assert rot_n == 0 or (cos.shape[1] == rot_n // 2 and sin.shape == cos.shape)
+    assert q_norm is None or q_norm.numel() == (d if head_norm else heads * d)
+    assert k_norm is None or k_norm.numel() == (d if head_norm else g * d)
     t = src.shape[0]
     q = torch.empty((t, heads * d), dtype=torch.float32, device=src.device)
     with _k("qk_norm_rope_kv_write"):
@@ -1139,7 +1151,7 @@ def qk_norm_rope_kv_write(src, q_col0: int, k_col0: int, v_col0: int, heads: int
                                                       float(eps), int(rot_n), 1 if rot_half else 0, _ptr(cos), _ptr(sin),
                                                       _ptr(meta.tok_pos), _ptr(meta.slot_mapping), _ptr(q), _ptr(k_pool),
                                                       _ptr(v_pool), _edt(k_pool), t, heads, g, gv, d, dv, bs, _ptr(q_head_scale),
-                                                      _stream()),
+                                                      1 if head_norm else 0, _stream()),
               "b200_qk_norm_rope_kv_write")
     return q
 
@@ -1234,4 +1246,126 @@ def gated_scan(proj, q_col0: int, f_col0: int, v_col0: int, f_bias, lower, state
                                   _ptr(meta.seq_slot), _ptr(meta.seq_pos0), _ptr(out), meta.num_seqs, heads, dim, vdim,
                                   _ptr(segs) if nseg else 0, nseg, _ptr(meta.scan_seq_seg0) if nseg else 0, _ptr(seg_state),
                                   _ptr(seg_decay), _stream()), "b200_gated_scan")
+    return out
+
+
+# ------------------------------------------------------------------ post-layer-norm decoders (selective scan, matrix memory)
+SEL_SEGS_MAX_CTAS = 592  # whole-portion CTAs of the selective scan (four per SM) below which long portions run as segments
+
+
+def selective_scan(x, dt_raw, bc, b_col0: int, c_col0: int, z, a_log2, dt_bias, d_skip, state, meta):
+    """Selective scan with a step size per channel: S[c, n] <- exp(dt A[c, n]) S[c, n] + dt x B[n], y = S . C + d_skip x, times
+    silu(z) when z is given.  x [T, C] (bf16 | fp32); dt_raw fp32 [T, C] (any pitch), dt = softplus(dt_raw + dt_bias); B / C = columns
+    b_col0 / c_col0 ([N] each) of the fp32 rows bc; z fp32 [T, C] view (any pitch) or None; a_log2 fp32 [C, N] = A log2(e);
+    state fp32 [slots, C, N] updated in place.  Returns y [T, C] in x's type."""
+    _cuda(x, dt_raw, bc, z, a_log2, dt_bias, d_skip, state)
+    _f32(a_log2, dt_bias, d_skip, state)
+    t, c = x.shape
+    n = a_log2.shape[1]
+    assert x.is_contiguous() and state.shape[1:] == (c, n) == a_log2.shape and dt_bias.numel() == c == d_skip.numel()
+    for r in (dt_raw, bc, z):
+        assert r is None or (r.dtype == torch.float32 and r.stride(1) == 1 and r.shape[0] == t)
+    assert dt_raw.shape[1] >= c and bc.shape[1] >= max(b_col0, c_col0) + n and (z is None or z.shape[1] >= c)
+    out = torch.empty_like(x)
+    segs = getattr(meta, "scan_segs", None)
+    nseg = meta.num_segs if segs is not None else 0
+    lanes = 4 if n <= 64 else 8 if n <= 128 else 16  # lanes that share a channel (256 threads per CTA)
+    if -(-c // (256 // lanes)) * meta.num_seqs >= SEL_SEGS_MAX_CTAS:
+        nseg = 0
+    seg_state = seg_dt = None
+    if nseg:
+        seg_state = torch.empty((nseg, c, n), dtype=torch.float32, device=x.device)
+        seg_dt = torch.empty((nseg, c), dtype=torch.float32, device=x.device)
+    with _k("selective_scan"):
+        check(_cabi.load().b200_selective_scan(_ptr(x), _edt(x), _ptr(dt_raw), dt_raw.stride(0), _ptr(bc), bc.stride(0), b_col0, c_col0,
+                                               _ptr(z), z.stride(0) if z is not None else 0, _ptr(a_log2), _ptr(dt_bias),
+                                               _ptr(d_skip), _ptr(state), _ptr(meta.seq_start), _ptr(meta.seq_slot),
+                                               _ptr(meta.seq_pos0), _ptr(out), meta.num_seqs, c, n, _ptr(segs) if nseg else 0, nseg,
+                                               _ptr(meta.scan_seq_seg0) if nseg else 0, _ptr(seg_state), _ptr(seg_dt), _stream()),
+              "b200_selective_scan")
+    return out
+
+
+def matrix_memory(proj, q_col0: int, k_col0: int, v_col0: int, i_col0: int, f_col0: int, i_bias, f_bias, cap: float, state, m_state,
+                  meta, heads: int, dim: int, vdim: int):
+    """Matrix memory with exponential input gates over a ragged batch: q / k / v and the raw gates are columns of the fp32 rows proj.
+    state fp32 [slots, H, vdim + 1, dim] (the last column is the normaliser) and m_state fp32 [slots, H] (running maximum) are
+    updated in place.  Returns (S^T q [T, H * vdim], n . q [T, H], exp(-m) [T, H]), q unscaled."""
+    _cuda(proj, i_bias, f_bias, state, m_state)
+    _f32(i_bias, f_bias, state, m_state)
+    assert proj.dtype == torch.float32 and proj.stride(1) == 1 and state.shape[1:] == (heads, vdim + 1, dim)
+    assert i_bias.numel() == heads == f_bias.numel() and m_state.shape[1:] == (heads,)
+    t = proj.shape[0]
+    coef = torch.empty((t, heads, 2), dtype=torch.float32, device=proj.device)
+    floor = torch.empty((t, heads), dtype=torch.float32, device=proj.device)
+    out = torch.empty((t, heads * vdim), dtype=torch.float32, device=proj.device)
+    out_n = torch.empty((t, heads), dtype=torch.float32, device=proj.device)
+    lib = _cabi.load()
+    with _k("matrix_memory_gates"):
+        check(lib.b200_matrix_memory_gates(_ptr(proj), proj.stride(0), i_col0, f_col0, _ptr(i_bias), _ptr(f_bias), float(cap),
+                                           _ptr(m_state), _ptr(meta.seq_start), _ptr(meta.seq_slot), _ptr(meta.seq_pos0), _ptr(coef),
+                                           _ptr(floor), meta.num_seqs, heads, _stream()), "b200_matrix_memory_gates")
+    segs = getattr(meta, "scan_segs", None)
+    nseg = meta.num_segs if segs is not None else 0
+    if -(-(vdim + 1) // 16) * heads * meta.num_seqs >= GATED_SEGS_MAX_CTAS:
+        nseg = 0
+    seg_state = seg_decay = None
+    if nseg:
+        seg_state = torch.empty((nseg, heads, vdim + 1, dim), dtype=torch.float32, device=proj.device)
+        seg_decay = torch.empty((nseg, heads, dim), dtype=torch.float32, device=proj.device)
+    with _k("matrix_memory_scan"):
+        check(lib.b200_matrix_memory_scan(_ptr(proj), proj.stride(0), q_col0, k_col0, v_col0, _ptr(coef), _ptr(state),
+                                          _ptr(meta.seq_start), _ptr(meta.seq_slot), _ptr(meta.seq_pos0), _ptr(out), _ptr(out_n),
+                                          meta.num_seqs, heads, dim, vdim, _ptr(segs) if nseg else 0, nseg,
+                                          _ptr(meta.scan_seq_seg0) if nseg else 0, _ptr(seg_state), _ptr(seg_decay), _stream()),
+              "b200_matrix_memory_scan")
+    return out, out_n, floor
+
+
+def matrix_memory_out(o, nq, floor, scale: float, gate_src, gate_col0: int, w, eps: float, heads: int, out_dtype):
+    """u = scale o / (max(|scale nq|, floor) + 1e-6) per head, then u / rms(u) * w * sigmoid(gate) -> [T, H * P] in out_dtype."""
+    _cuda(o, nq, floor, gate_src, w)
+    _f32(o, nq, floor, w)
+    assert gate_src.dtype == torch.float32 and gate_src.stride(1) == 1
+    t, hp = o.shape
+    assert w.numel() == hp
+    out = torch.empty((t, hp), dtype=out_dtype, device=o.device)
+    with _k("matrix_memory_out"):
+        check(_cabi.load().b200_matrix_memory_out(_ptr(o), _ptr(nq), _ptr(floor), float(scale), _ptr(gate_src), gate_src.stride(0),
+                                                  gate_col0, _ptr(w), float(eps), _ptr(out), _edt(out), t, heads, hp // heads,
+                                                  _stream()), "b200_matrix_memory_out")
+    return out
+
+
+def postln_residual(x, alpha: float, w, eps: float, *, y1=None, w1=None, y2=None, w2=None, c: float = 1.0, vec=None, out_dtype=None,
+                    store: bool = True):
+    """u = alpha x + vec + c (N(y1) w1 + N(y2) w2) with N = division by the row's RMS (y2 None: u = alpha x + vec + c y1, every term
+    optional), then a layer norm without bias: (u - mean) / sqrt(var + eps) * w -> x in place (store) and, in out_dtype, the
+    returned rows (None without out_dtype)."""
+    _cuda(x, w, y1, w1, y2, w2, vec)
+    _f32(x, w, w1, w2, vec)
+    t, width = x.shape
+    for y in (y1, y2):
+        assert y is None or (y.dtype == torch.float32 and y.stride(1) == 1 and y.shape == (t, width))
+    assert w.numel() == width and (vec is None or vec.numel() == width)
+    out = torch.empty((t, width), dtype=out_dtype, device=x.device) if out_dtype is not None else None
+    with _k("postln_residual"):
+        check(_cabi.load().b200_postln_residual(_ptr(x), float(alpha), _ptr(y1), y1.stride(0) if y1 is not None else 0, _ptr(w1),
+                                                _ptr(y2), y2.stride(0) if y2 is not None else 0, _ptr(w2), float(c), _ptr(vec),
+                                                _ptr(w), float(eps), 1 if store else 0, _ptr(out),
+                                                _edt(out_dtype) if out_dtype is not None else F32, t, width, _stream()),
+              "b200_postln_residual")
+    return out
+
+
+def bias_act(src, col0: int, n: int, bias, act: int, out_dtype):
+    """act(columns [col0, col0 + n) of the fp32 rows src + bias) -> [T, n] in out_dtype; act = ACT_NONE | ACT_RELU2; bias may be None."""
+    _cuda(src, bias)
+    _f32(bias)
+    assert src.dtype == torch.float32 and src.stride(1) == 1 and (bias is None or bias.numel() == n)
+    t = src.shape[0]
+    out = torch.empty((t, n), dtype=out_dtype, device=src.device)
+    with _k("bias_act"):
+        check(_cabi.load().b200_bias_act(_ptr(src), src.stride(0), col0, n, _ptr(bias), int(act), _ptr(out), _edt(out), t, _stream()),
+              "b200_bias_act")
     return out

@@ -9,7 +9,9 @@ Two families are served:
     bigram embedding, dense or MoE feed-forward; "Zudarax": parallel mixer / feed-forward branches behind one grouped RMS
     norm, three rotating-attention variants (chunked + soft-capped, differential, sigmoid), polynomial activation;
     "Gerupel": parallel branches behind two RMS norms, a mixer that is windowed attention with pooled far blocks beside a gated
-    linear recurrence, repeated layer runs with shared weights, MoE, logits from the embedding table.
+    linear recurrence, repeated layer runs with shared weights, MoE, logits from the embedding table; "Goponex": layer norm after
+    the sum, a mixer that is windowed attention with kept first tokens (values = keys) beside a selective scan with a step size per
+    channel, matrix-memory layers, squared-relu feed-forward.
 The reference resolves the architecture the same way -- `hf_config.architectures[0]` picks the NxDI model class
 (vllm_neuron/worker/neuronx_distributed_model_loader.py:612-660).
 """
@@ -79,6 +81,7 @@ MODEL_REGISTRY: dict[str, ModelEntry] = {
     "Kenetar": ModelEntry("hybrid", _hybrid_config, _hybrid_weights, _hybrid_build, (torch.bfloat16, torch.float32)),
     "Zudarax": ModelEntry("hybrid", _hybrid_config, _hybrid_weights, _hybrid_build, (torch.bfloat16, torch.float32)),
     "Gerupel": ModelEntry("hybrid", _hybrid_config, _hybrid_weights, _hybrid_build, (torch.bfloat16, torch.float32)),
+    "Goponex": ModelEntry("hybrid", _hybrid_config, _hybrid_weights, _hybrid_build, (torch.bfloat16, torch.float32)),
 }
 
 

@@ -527,11 +527,12 @@ int b200_matrix_memory_out(const float* o, const float* nq, const float* floor_i
  * y_c = sum_n S[c][n] C_n + d_skip_c x_c, out = y silu(z) (z NULL: y).  x, out [T][C] in x_dtype; dt = softplus(dt_raw + dt_bias);
  * B, C = columns b_col0 / c_col0 ([N] each) of the fp32 rows bc; a_log2 fp32 [C][N] = A log2(e); state fp32 [slots][C][N], read when
  * seq_pos0 > 0, written back for all.  num_segs > 0: segments as in b200_gated_scan, scratch seg_state fp32 [num_segs][C][N] and
- * seg_dt fp32 [num_segs][C].  N <= 256, else B200_ERR_UNSUPPORTED. */
+ * seg_dt fp32 [num_segs][C].  max_new: the longest portion of the step (picks the kernel; any value not below it is correct).  N <= 256, else B200_ERR_UNSUPPORTED. */
 int b200_selective_scan(const void* x, int x_dtype, const float* dt_raw, int ld_dt, const float* bc, int ld_bc, int b_col0, int c_col0,
                         const float* z, int ld_z, const float* a_log2, const float* dt_bias, const float* d_skip, float* state,
                         const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_pos0, void* out, int B, int C, int N,
-                        const int32_t* segs, int num_segs, const int32_t* seq_seg0, float* seg_state, float* seg_dt, void* stream);
+                        const int32_t* segs, int num_segs, const int32_t* seq_seg0, float* seg_state, float* seg_dt, int max_new,
+                        void* stream);
 /* Post-norm residual step with a layer norm: u = alpha x + [vec +] c (N(y1) w1 + N(y2) w2), N = division by the row's RMS (y2 NULL:
  * u = alpha x + [vec +] c y1, y1 may be NULL too);  x (when store_x) = out (when given) = (u - mean) / sqrt(var + eps) * w. */
 int b200_postln_residual(float* x, float alpha, const float* y1, int ld1, const float* w1, const float* y2, int ld2, const float* w2,

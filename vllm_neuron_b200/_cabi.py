@@ -120,7 +120,7 @@ SIGNATURES = {
     "b200_matrix_memory_scan": (_i, [_p, _i, _i, _i, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _p, _i, _p, _p, _p, _p]),
     "b200_matrix_memory_out": (_i, [_p, _p, _p, _f, _p, _i, _i, _p, _f, _p, _i, _i, _i, _i, _p]),
     "b200_selective_scan": (_i, [_p, _i, _p, _i, _p, _i, _i, _i, _p, _i, _p, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _p, _i, _p, _p, _p,
-                                 _p]),
+                                 _i, _p]),
     "b200_postln_residual": (_i, [_p, _f, _p, _i, _p, _p, _i, _p, _f, _p, _p, _f, _i, _p, _i, _i, _i, _p]),
     "b200_bias_act": (_i, [_p, _i, _i, _i, _p, _i, _p, _i, _i, _p]),
     "b200_delta_prep": (_i, [_p, _i, _p, _i, _i, _i, _p, _p, _p, _p, _i, _i, _i, _i, _f, _f, _p]),

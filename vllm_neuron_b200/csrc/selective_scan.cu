@@ -14,6 +14,8 @@
 //     S_end = exp(A sum dt) S0 + Z_end: the PARTIAL pass leaves Z_end and sum dt of every segment but a sequence's last, an
 //     elementwise pass chains them, the FULL pass runs every segment from its true start state.  The recurrence is linear in S:
 //     this is the sequential result up to fp32 rounding.
+//   * steps whose portions are all short (decoding): a kernel without staging -- every operand goes straight to registers, one
+//     dependent round of loads, no barrier; same arithmetic in the same order.
 // State layout [slots][C][N].  A sequence whose portion starts at position 0 ignores what its slot held.
 #include "hybrid_common.cuh"
 
@@ -21,6 +23,7 @@ namespace b200 {
 
 constexpr int SEL_THREADS = 256;
 constexpr int SEL_CHUNK = 16;  // tokens staged per round
+constexpr int SEL_STEP_TOKENS = 4;  // longest portion of a step that runs without staging
 
 __device__ __forceinline__ float sel_ex2(float x) {
   float y;
@@ -203,6 +206,81 @@ __global__ void __launch_bounds__(SEL_THREADS)
   if (MODE == 1 && r == 0 && live) seg_dt[(int64_t)blockIdx.y * C + c] = dsum;
 }
 
+// Short portions: LPC lanes per channel as above, operands straight from memory; bvec = B and C rows on the 16-byte grid.
+template <typename XT, typename OT, int LPC, int NPT>
+__global__ void __launch_bounds__(SEL_THREADS)
+    selective_step_kernel(const XT* __restrict__ x, const float* __restrict__ dt_raw, int ld_dt, const float* __restrict__ bc, int ld_bc,
+                          int b_col0, int c_col0, const float* __restrict__ z, int ld_z, const float* __restrict__ a_log2,
+                          const float* __restrict__ dt_bias, const float* __restrict__ d_skip, float* __restrict__ state,
+                          const int32_t* __restrict__ seq_start, const int32_t* __restrict__ seq_slot,
+                          const int32_t* __restrict__ seq_pos0, OT* __restrict__ out, int C, int N, int bvec) {
+  griddep_launch();
+  const int idx = blockIdx.x * SEL_THREADS + threadIdx.x, r = idx % LPC, c = idx / LPC, sq = blockIdx.y;
+  const bool live = c < C, vec = (N & 3) == 0;
+  const int cc = live ? c : 0;
+  auto ld4s = [&](const float* p, int n, bool v4) -> float4 {
+    if (v4) return n < N ? *reinterpret_cast<const float4*>(p + n) : make_float4(0.f, 0.f, 0.f, 0.f);
+    return make_float4(n < N ? p[n] : 0.f, n + 1 < N ? p[n + 1] : 0.f, n + 2 < N ? p[n + 2] : 0.f, n + 3 < N ? p[n + 3] : 0.f);
+  };
+  // what no kernel of the step writes: decay rates, bias, skip
+  float2 S[NPT / 2], A[NPT / 2];
+  const float* ar = a_log2 + (int64_t)cc * N;
+#pragma unroll
+  for (int k = 0; k < NPT / 4; ++k) {
+    const float4 a = ld4s(ar, 4 * (r + LPC * k), vec);
+    A[2 * k] = make_float2(a.x, a.y), A[2 * k + 1] = make_float2(a.z, a.w);
+  }
+  const float bias = dt_bias[cc], skip = d_skip[cc];
+  griddep_wait();
+  const int t0 = seq_start[sq], t1 = seq_start[sq + 1];
+  if (t0 >= t1) return;
+  float* slot = state + ((int64_t)seq_slot[sq] * C + cc) * N;
+  const bool cont = seq_pos0[sq] > 0;
+#pragma unroll
+  for (int k = 0; k < NPT / 4; ++k) {
+    const float4 s = cont ? ld4s(slot, 4 * (r + LPC * k), vec) : make_float4(0.f, 0.f, 0.f, 0.f);
+    S[2 * k] = make_float2(s.x, s.y), S[2 * k + 1] = make_float2(s.z, s.w);
+  }
+  for (int64_t t = t0; t < t1; ++t) {
+    const float v = dt_raw[t * ld_dt + cc] + bias, xv = ldf(x, t * C + cc), zv = z ? z[t * ld_z + cc] : 0.f;
+    const float dt = v > 20.f ? v : log1pf(expf(v)), dx = dt * xv;
+    const float2 dt2 = make_float2(dt, dt), dx2 = make_float2(dx, dx);
+    const float* row = bc + t * ld_bc;
+    float2 acc = make_float2(0.f, 0.f);
+#pragma unroll
+    for (int k = 0; k < NPT / 4; ++k) {
+      const float4 b4 = ld4s(row + b_col0, 4 * (r + LPC * k), bvec), c4 = ld4s(row + c_col0, 4 * (r + LPC * k), bvec);
+      const float2 e0 = fmul2(dt2, A[2 * k]), e1 = fmul2(dt2, A[2 * k + 1]);
+      const float2 g0 = make_float2(sel_ex2(e0.x), sel_ex2(e0.y)), g1 = make_float2(sel_ex2(e1.x), sel_ex2(e1.y));
+      S[2 * k] = ffma2(g0, S[2 * k], fmul2(dx2, make_float2(b4.x, b4.y)));
+      S[2 * k + 1] = ffma2(g1, S[2 * k + 1], fmul2(dx2, make_float2(b4.z, b4.w)));
+      acc = ffma2(S[2 * k], make_float2(c4.x, c4.y), acc);
+      acc = ffma2(S[2 * k + 1], make_float2(c4.z, c4.w), acc);
+    }
+    float y = acc.x + acc.y;
+#pragma unroll
+    for (int o = 1; o < LPC; o <<= 1) y += __shfl_xor_sync(0xffffffffu, y, o);
+    if (r == 0 && live) {
+      y += skip * xv;
+      if (z) y *= silu_f(zv);
+      stf(out, t * C + cc, y);
+    }
+  }
+  if (!live) return;
+#pragma unroll
+  for (int k = 0; k < NPT / 4; ++k) {
+    const int n = 4 * (r + LPC * k);
+    if (vec) {
+      if (n < N) *reinterpret_cast<float4*>(slot + n) = make_float4(S[2 * k].x, S[2 * k].y, S[2 * k + 1].x, S[2 * k + 1].y);
+    } else {
+      if (n < N) slot[n] = S[2 * k].x;
+      if (n + 1 < N) slot[n + 1] = S[2 * k].y;
+      if (n + 2 < N) slot[n + 2] = S[2 * k + 1].x;
+      if (n + 3 < N) slot[n + 3] = S[2 * k + 1].y;
+    }
+  }
+}
+
 // Chains the segments of every sequence, one thread per state element: segment k's entry of seg_state (Z_end) is replaced by its
 // START state; carry <- 2^(A sum_dt[k]) carry + Z_end[k].
 __global__ void selective_seg_combine_kernel(const float* __restrict__ state, float* __restrict__ seg_state,
@@ -244,7 +322,14 @@ static int launch_selective(const void* x, const float* dt_raw, int ld_dt, const
                             const float* z, int ld_z, const float* a_log2, const float* dt_bias, const float* d_skip, float* state,
                             const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_pos0, void* out, int B, int C, int N,
                             const int32_t* segs, int num_segs, const int32_t* seq_seg0, float* seg_state, float* seg_dt,
-                            cudaStream_t st) {
+                            int max_new, cudaStream_t st) {
+  if (num_segs == 0 && max_new <= SEL_STEP_TOKENS) {
+    const int bvec = (N & 3) == 0 && ld_bc % 4 == 0 && b_col0 % 4 == 0 && c_col0 % 4 == 0 && ((uintptr_t)bc & 15) == 0;
+    B200_CUDA_OK(launch_kernel(selective_step_kernel<XT, OT, LPC, NPT>, dim3((unsigned)(((int64_t)C * LPC + SEL_THREADS - 1) / SEL_THREADS), B),
+                               dim3(SEL_THREADS), 0, st, (const XT*)x, dt_raw, ld_dt, bc, ld_bc, b_col0, c_col0, z, ld_z, a_log2, dt_bias,
+                               d_skip, state, seq_start, seq_slot, seq_pos0, (OT*)out, C, N, bvec));
+    return B200_OK;
+  }
   const unsigned gx = (C + SEL_THREADS / LPC - 1) / (SEL_THREADS / LPC);
   const int4* sg = reinterpret_cast<const int4*>(segs);
 #define SEL_GO(MODE, LAUNCH, NY)                                                                                                 \
@@ -275,7 +360,8 @@ extern "C" {
 int b200_selective_scan(const void* x, int x_dtype, const float* dt_raw, int ld_dt, const float* bc, int ld_bc, int b_col0, int c_col0,
                         const float* z, int ld_z, const float* a_log2, const float* dt_bias, const float* d_skip, float* state,
                         const int32_t* seq_start, const int32_t* seq_slot, const int32_t* seq_pos0, void* out, int B, int C, int N,
-                        const int32_t* segs, int num_segs, const int32_t* seq_seg0, float* seg_state, float* seg_dt, void* stream) {
+                        const int32_t* segs, int num_segs, const int32_t* seq_seg0, float* seg_state, float* seg_dt, int max_new,
+                        void* stream) {
   B200_REQUIRE(x && dt_raw && bc && a_log2 && dt_bias && d_skip && state && seq_start && seq_slot && seq_pos0 && out,
                "selective_scan: null pointer");
   B200_REQUIRE(C >= 1 && N >= 1, "selective_scan: bad shape");
@@ -293,7 +379,7 @@ int b200_selective_scan(const void* x, int x_dtype, const float* dt_raw, int ld_
 #define SEL_PICK(LPC, NPT)                                                                                                         \
   return launch_selective<XT, XT, LPC, NPT>(x, dt_raw, ld_dt, bc, ld_bc, b_col0, c_col0, z, ld_z, a_log2, dt_bias, d_skip, state, \
                                             seq_start, seq_slot, seq_pos0, out, B, C, N, segs, num_segs, seq_seg0, seg_state,     \
-                                            seg_dt, st)
+                                            seg_dt, max_new, st)
   B200_DISPATCH_ELEM(x_dtype, XT, {
     if (N <= 16) SEL_PICK(4, 4);
     if (N <= 32) SEL_PICK(4, 8);

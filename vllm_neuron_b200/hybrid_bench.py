@@ -1,7 +1,9 @@
 """Prefill / decode throughput of the hybrid decoders (bench.py --hybrid): the Pumopel design next to the dense Llama decoder
 at equal size (`small`, `1b`), the Kenetar design next to Pumopel at equal size (`kenetar-small`, `kenetar-1b`), the
 Zudarax design next to the dense Llama decoder at equal size (`zudarax-small`, `zudarax-1b`), and the Gerupel design next to
-Pumopel (its closest relative: windowed sink attention, a recurrence, experts) at equal size (`gerupel-small`, `gerupel-1b`).
+Pumopel (its closest relative: windowed sink attention, a recurrence, experts) at equal size (`gerupel-small`, `gerupel-1b`),
+and the Goponex design next to Gerupel (windowed attention beside a recurrence) and Pumopel (a state-space scan) at equal size
+(`goponex-small`, `goponex-1b`).
 
 For each size: random weights, both models in bf16 on one GPU, same width / layer count / vocabulary; the dense model's
 intermediate size equals the hybrid's ACTIVE feed-forward width (top * ff + shared ff) so a token costs about the same FLOPs.
@@ -107,6 +109,63 @@ def _gerupel_floors(name, t, s_pre, ctx, b, prefill):
         "moe_gate_up_glu": (4.0 * npairs * gm["ff"] * w, used * 4.0 * gm["ff"] * w + t * 2 * w + npairs * 2 * gm["ff"]),
         "moe_down": (2.0 * npairs * gm["ff"] * w, used * 2.0 * gm["ff"] * w + npairs * (2 * gm["ff"] + 4 * w)),
         "moe_gather_scale": (0.0, npairs * w * 4.0),
+    })
+    return out
+
+
+# the layer-norm-after-the-sum design at the same width / layers / vocabulary / attention sizes: layer pattern 'p p m p' repeated
+# (p: windowed attention with kept tokens beside a selective scan of twice the width; m: matrix memory with as many state
+# elements as Gerupel's recurrence, no feed-forward); squared-relu feed-forward of two matrices with as many weights as the
+# hybrid's active three
+GOPONEX_MIXERS = {
+    "1b": dict(keep=4, right=dict(inner=4096, state=16, dt_rank=128, conv=4), mlstm=dict(heads=8, dim=128, vdim=256, gate_cap=15.0)),
+    "small": dict(keep=4, right=dict(inner=2048, state=16, dt_rank=64, conv=4), mlstm=dict(heads=8, dim=64, vdim=128, gate_cap=15.0)),
+}
+
+
+def _goponex_ff(sz):
+    return 3 * (sz["moe"]["top"] * sz["moe"]["ff"] + sz["moe"]["shared"]) // 2
+
+
+def goponex_config(name: str):
+    from .hybrid import HybridConfig
+
+    sz, gm = SIZES[name], GOPONEX_MIXERS[name]
+    a = sz["attn"]
+    yarn = {"factor": 8.0, "original": 4096, "fast": 32.0, "slow": 1.0}
+    left = {"heads": a["heads"], "kv_heads": a["kv_heads"], "dim": a["dim"], "vdim": a["dim"], "scale": a["dim"] ** -0.5,
+            "rot": {"dims": a["dim"] // 2, "base": 500000.0, "scaling": yarn}, "mask": {"size": a["window"], "keep_first": gm["keep"]}}
+    par = {"type": "parallel", "mixer": {"left": left, "right": dict(gm["right"])}, "mlp": {"kind": "dense", "ff": _goponex_ff(sz)}}
+    mem = {"type": "mlstm", "mixer": dict(gm["mlstm"]), "mlp": None}
+    return HybridConfig.from_dict({"architecture": "Goponex", "vocab": sz["vocab"], "width": sz["width"], "norm": {"eps": 1e-6},
+                                   "postln_alpha": 2.0, "layers": [mem if i % 4 == 2 else par for i in range(sz["layers"])]})
+
+
+def _goponex_floors(name, t, s_pre, ctx, b, prefill):
+    """Algorithmic (flops, bytes) per launch of the layer-norm-after-the-sum design's own kernels at `t` tokens."""
+    sz, gm = SIZES[name], GOPONEX_MIXERS[name]
+    a, r, m, w = sz["attn"], gm["right"], gm["mlstm"], sz["width"]
+    h, g, d, win, keep = a["heads"], a["kv_heads"], a["dim"], a["window"], gm["keep"]
+    seen = lambda i: min(i + 1, win) + min(keep, max(0, i + 1 - win))  # noqa: E731  keys that position i sees
+    if prefill:
+        pairs_qk, kv_rows, nseq = float(sum(seen(i) for i in range(s_pre))), s_pre, 1
+    else:
+        pairs_qk, kv_rows, nseq = float(b * seen(ctx)), b * seen(ctx), b
+    att = (4.0 * h * pairs_qk * d, 4.0 * kv_rows * g * d + t * h * 6.0 * d)
+    hd, hp, ff = m["heads"] * m["dim"], m["heads"] * m["vdim"], _goponex_ff(sz)
+    mm_state = m["heads"] * m["dim"] * (m["vdim"] + 1)
+    out = {k + "[keep]": att for k in ("swa_sink_attn_prefill", "swa_sink_attn_prefill_tc", "swa_sink_attn", "swa_sink_attn_decode_tc")}
+    out.update({
+        "selective_scan": (6.0 * t * r["inner"] * r["state"],
+                           t * (12.0 * r["inner"] + 8.0 * r["state"]) + 8.0 * nseq * r["inner"] * r["state"] + 4.0 * r["inner"] * r["state"]),
+        "matrix_memory_scan": (6.0 * t * mm_state, t * 4.0 * (2 * hd + 2 * hp) + 8.0 * nseq * mm_state),
+        "matrix_memory_gates": (0.0, t * m["heads"] * 20.0),
+        "matrix_memory_out": (0.0, t * hp * 10.0),
+        "causal_conv_silu": (0.0, t * r["inner"] * 6.0),
+        "qk_norm_rope_kv_write": (0.0, t * (4.0 * (h + g) * d + 4.0 * h * d + 4.0 * g * d)),
+        "postln_residual": (0.0, t * w * 14.0), "postln_residual[2]": (0.0, t * w * 18.0),
+        "bias_act[relu2]": (0.0, t * ff * 6.0), "bias_act": (0.0, t * r["dt_rank"] * 6.0),
+        "embed_bigram": (0.0, t * w * 8.0),
     })
     return out
 
@@ -352,12 +411,13 @@ def run(args):
     names = list(SIZES) if args.hybrid == "all" else [args.hybrid]
     for name in names:
         kenetar, zudarax, gerupel = name.startswith("kenetar-"), name.startswith("zudarax-"), name.startswith("gerupel-")
-        short = name.split("-", 1)[1] if kenetar or zudarax or gerupel else name
+        goponex = name.startswith("goponex-")
+        short = name.split("-", 1)[1] if kenetar or zudarax or gerupel or goponex else name
         sz = SIZES[short]
         cfg = hybrid_config(sz)
         s_pre, b, ctx = sz["prefill"], sz["batch"], sz["ctx"]
         bs = 32
-        res = {"metric": "gerupel_vs_pumopel_tokens_per_s" if gerupel else "kenetar_vs_pumopel_tokens_per_s" if kenetar else "zudarax_vs_dense_tokens_per_s" if zudarax else
+        res = {"metric": "goponex_vs_gerupel_tokens_per_s" if goponex else "gerupel_vs_pumopel_tokens_per_s" if gerupel else "kenetar_vs_pumopel_tokens_per_s" if kenetar else "zudarax_vs_dense_tokens_per_s" if zudarax else
                "hybrid_vs_dense_tokens_per_s", "size": name,
                "dtype": "bf16", "data": "synthetic (random weights)",
                "roofline_peaks": {"hbm_gbs": hbm / 1e9, "bf16_tflops": peak / 1e12, "source": src},
@@ -366,6 +426,15 @@ def run(args):
         win = sz["attn"]["window"]
         pum_floors = lambda t, pre: _floors(cfg, sz, t, min(win, s_pre / 2) if pre else min(win, ctx + 1),  # noqa: E731
                                             s_pre if pre else b * min(win, ctx + 1), 1 if pre else b)
+        if goponex:
+            gop_floors = lambda t, pre: _goponex_floors(short, t, s_pre, ctx, b, pre)  # noqa: E731
+            ger_floors = lambda t, pre: _gerupel_floors(short, t, s_pre, ctx, b, pre)  # noqa: E731
+            res["goponex"] = _time_hybrid(goponex_config(short), sz, args, gop_floors, flush, hbm, peak)[0]
+            res["gerupel"] = _time_hybrid(gerupel_config(short), sz, args, ger_floors, flush, hbm, peak)[0]
+            res["pumopel"] = _time_hybrid(cfg, sz, args, pum_floors, flush, hbm, peak)[0]
+            res["gpu_launches"] = ops.launch_count()
+            print(json.dumps(res), flush=True)
+            continue
         if gerupel:
             ger_floors = lambda t, pre: _gerupel_floors(short, t, s_pre, ctx, b, pre)  # noqa: E731
             res["gerupel"] = _time_hybrid(gerupel_config(short), sz, args, ger_floors, flush, hbm, peak)[0]

@@ -1281,7 +1281,7 @@ def selective_scan(x, dt_raw, bc, b_col0: int, c_col0: int, z, a_log2, dt_bias, 
                                                _ptr(z), z.stride(0) if z is not None else 0, _ptr(a_log2), _ptr(dt_bias),
                                                _ptr(d_skip), _ptr(state), _ptr(meta.seq_start), _ptr(meta.seq_slot),
                                                _ptr(meta.seq_pos0), _ptr(out), meta.num_seqs, c, n, _ptr(segs) if nseg else 0, nseg,
-                                               _ptr(meta.scan_seq_seg0) if nseg else 0, _ptr(seg_state), _ptr(seg_dt), _stream()),
+                                               _ptr(meta.scan_seq_seg0) if nseg else 0, _ptr(seg_state), _ptr(seg_dt), meta.max_new, _stream()),
               "b200_selective_scan")
     return out
 
@@ -1349,7 +1349,7 @@ def postln_residual(x, alpha: float, w, eps: float, *, y1=None, w1=None, y2=None
         assert y is None or (y.dtype == torch.float32 and y.stride(1) == 1 and y.shape == (t, width))
     assert w.numel() == width and (vec is None or vec.numel() == width)
     out = torch.empty((t, width), dtype=out_dtype, device=x.device) if out_dtype is not None else None
-    with _k("postln_residual"):
+    with _k("postln_residual[2]" if y2 is not None else "postln_residual"):
         check(_cabi.load().b200_postln_residual(_ptr(x), float(alpha), _ptr(y1), y1.stride(0) if y1 is not None else 0, _ptr(w1),
                                                 _ptr(y2), y2.stride(0) if y2 is not None else 0, _ptr(w2), float(c), _ptr(vec),
                                                 _ptr(w), float(eps), 1 if store else 0, _ptr(out),
@@ -1365,7 +1365,7 @@ def bias_act(src, col0: int, n: int, bias, act: int, out_dtype):
     assert src.dtype == torch.float32 and src.stride(1) == 1 and (bias is None or bias.numel() == n)
     t = src.shape[0]
     out = torch.empty((t, n), dtype=out_dtype, device=src.device)
-    with _k("bias_act"):
+    with _k("bias_act[relu2]" if act == ACT_RELU2 else "bias_act"):
         check(_cabi.load().b200_bias_act(_ptr(src), src.stride(0), col0, n, _ptr(bias), int(act), _ptr(out), _edt(out), t, _stream()),
               "b200_bias_act")
     return out

@@ -1073,10 +1073,12 @@ class HybridCausalLM:
     def _linear(self, a, w):
         """fp32 [M, N] = a @ w^T.  bf16 serving: the tcgen05 GEMM (TMA needs K * 2 bytes to be a multiple of 16); anything
         else, and all of 32-bit serving, runs on the CUDA cores with true fp32 arithmetic.  A prompt-sized batch against a
-        very narrow weight (the router) would leave the 128-row tcgen05 weight tile almost empty: it takes the mma.sync
-        kernel behind linear_simt instead."""
-        if self.et == torch.bfloat16 and w.shape[1] % 8 == 0 and not (w.shape[0] <= 32 and a.shape[0] > 128):
-            m, (n, k) = a.shape[0], w.shape
+        very narrow weight (the router) would leave the 128-row tcgen05 weight tile almost empty, and one whose 256 x 128 output
+        tiles are few (narrow projections) would cut every tile's K range over many CTAs and wait for their fix-up: these, and
+        very short rows (all epilogue), take the mma.sync kernel behind linear_simt instead."""
+        m, (n, k) = a.shape[0], w.shape
+        narrow = m > 128 and (n <= 32 or k <= 128 or (n <= 256 and -(-m // 256) * -(-n // 128) <= 16))
+        if self.et == torch.bfloat16 and k % 8 == 0 and not narrow:
             need = ops.gemm_workspace_bytes(m, n, k, ops.BF16, 0)
             if need and (self.gemm_ws is None or self.gemm_ws.numel() < need):
                 self.gemm_ws = torch.zeros(need, dtype=torch.uint8, device=self.device)  # stream-K counters start at zero

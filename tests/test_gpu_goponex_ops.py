@@ -290,7 +290,7 @@ PAGES = {s: list(range(1 + 200 * s, 200 + 200 * s)) for s in range(4)}
 
 
 @pytest.mark.parametrize("x_dtype", [torch.float32, torch.bfloat16])
-@pytest.mark.parametrize("C,N,lead", [(10, 3, 1), (70, 16, 0), (256, 24, 4), (33, 64, 2), (130, 20, 0), (20, 100, 0), (17, 200, 3), (8, 256, 0), (5, 1, 0)])
+@pytest.mark.parametrize("C,N,lead", [(10, 3, 1), (70, 16, 0), (244, 24, 4), (33, 64, 2), (130, 20, 0), (20, 100, 0), (17, 200, 3), (8, 256, 0), (5, 1, 0)])
 @pytest.mark.parametrize("lens,steps", [SHORT, LONG], ids=["short", "segments"])
 def test_selective_scan_over_portions_slots_and_reuse(C, N, lead, x_dtype, lens, steps):
     """Raw step sizes and gate -> scan with gate, for sequences cut into portions beside each other (also steps of one to three

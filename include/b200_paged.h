@@ -33,7 +33,7 @@
 extern "C" {
 #endif
 
-#define B200_ABI_VERSION 13
+#define B200_ABI_VERSION 14
 
 enum {
   B200_OK = 0,
@@ -405,18 +405,24 @@ int b200_attn_split_merge(const float* part, int splits, int Dv, int sigmoid, in
  * heads.  v_col0 may equal k_col0 (the values are the keys as projected).  The first rot_n columns of every q and k head turn by tok_pos[t]: pairs (i, i + rot_n / 2) when
  * rot_half, else (2i, 2i + 1); (u, v) -> (u cos - v sin, v cos + u sin), cos / sin fp32 tables [positions][rot_n / 2].
  * q -> q_out fp32 [T][H * D], head h times q_head_scale[h] when given (a per-head temperature of the scores);
+ * bias (or NULL) fp32 [q: H * D | k: G * D | v: Gv * Dv]: the projections' biases, added first;
  * k, v -> pools K [num_blocks][G][block_size][D], V [num_blocks][Gv][block_size][Dv] by slot. */
 int b200_qk_norm_rope_kv_write(const float* src, int ld, int q_col0, int k_col0, int v_col0, const float* q_norm,
                                const float* k_norm, float eps, int rot_n, int rot_half, const float* cos_table,
                                const float* sin_table, const int32_t* tok_pos, const int64_t* slot_mapping, float* q_out,
                                void* k_pool, void* v_pool, int kv_dtype, int T, int H, int G, int Gv, int D, int Dv, int block_size,
-                               const float* q_head_scale, int head_norm, void* stream);
+                               const float* q_head_scale, int head_norm, const float* bias, void* stream);
 /* Router decision over fp32 logits [T] rows of pitch ld (+ bias fp32 [E] when given): the `top` largest (ties to the lower
  * index); weights = sigmoid of each chosen logit, no renormalisation (B200_ROUTE_SIGMOID), or the softmax over the chosen
  * logits only (B200_ROUTE_SOFTMAX_TOP), or the softmax over ALL experts with the chosen scores divided by their sum + 1e-20
  * (B200_ROUTE_SOFTMAX_RENORM). */
 int b200_moe_topk(const float* logits, int ld, const float* bias, int mode, int32_t* topk_idx, float* topk_weight, int T, int E,
                   int top, void* stream);
+/* Grouped router: s = softmax over all E experts, choice = s + correction (or NULL); the experts form `groups` equal runs of
+ * neighbours ranked by their largest choice score, only the experts of the best `keep` runs are eligible; the `top` largest
+ * choice scores win (ties to the lower index), weights = s * scale (without the correction, not renormalised). */
+int b200_moe_topk_grouped(const float* logits, int ld, const float* correction, int groups, int keep, float scale, int32_t* topk_idx,
+                          float* topk_weight, int T, int E, int top, void* stream);
 /* rows per expert tile of b200_moe_align / b200_grouped_linear; four times as many (tile_rows = 4 x this) are taken for
  * prompt-sized batches of 16-byte aligned bf16 operands, where every weight tile then serves 128 rows */
 int b200_moe_tile_rows(void);
@@ -441,10 +447,11 @@ int b200_grouped_linear(const void* a, int lda, const int32_t* sorted_ids, int g
                         void* stream);
 /* `batch` dense linears in one launch: out_b [M][N] = A_b [M][K] W_b [N][K]^T with A_b = a + b * a_batch_stride (pitch lda),
  * W_b = w + b * w_batch_stride, out_b = out + b * out_batch_stride (pitch ldo); fp32 accumulation.  The result is
- * multiplied by sigmoid(gate[row * gate_ld + b]) when gate != NULL and stored as fp32, or in `dtype` when out_typed. */
+ * multiplied by sigmoid(gate[row * gate_ld + b]) when gate != NULL (gate_cols: by sigmoid(gate[row * gate_ld + b * N + n]), a gate per
+ * output column) and stored as fp32, or in `dtype` when out_typed. */
 int b200_batched_linear(const void* a, int lda, int64_t a_batch_stride, const void* w, int64_t w_batch_stride, void* out, int ldo,
                         int64_t out_batch_stride, int batch, int M, int N, int K, int dtype, int out_typed, const float* gate,
-                        int gate_ld, void* stream);
+                        int gate_ld, int gate_cols, void* stream);
 
 /* ---------------------------------------------------------------- post-norm hybrid decoders (delta rule + latent attention)
  * x = table[token] * scale (+ bigram[row] when a bigram table is given: row = (prev * mul_prev + token * mul_cur) mod buckets,
@@ -571,8 +578,20 @@ int b200_latent_q_prep(const float* q, int ldq, int H, int D, int R, int rot_n, 
  * table row tok_row[t]) attends cache rows 0..pos; q fp32 [T][H][D] (pitch ldq), rows [D] with the values in the first Dv
  * columns; out bf16 [T][H][Dv].  D and Dv multiples of 16, Dv <= 256, else B200_ERR_UNSUPPORTED. */
 int b200_latent_attn_decode(const float* q, int ldq, const void* pool, const int32_t* block_table, int64_t bt_stride,
-                            const int32_t* tok_row, const int32_t* tok_pos, float scale, void* out, int T, int H, int D, int Dv,
-                            int block_size, void* stream);
+                            const int32_t* tok_row, const int32_t* tok_pos, const float* sink, float scale, int window, void* out,
+                            int T, int H, int D, int Dv, int block_size, void* stream);
+
+/* ---------------------------------------------------------------- hyper-connections
+ * The residual stream of a token is S copies (x fp32 [T][S][W], S <= 32).  hyper_embed: every copy = table[token];
+ * out (dtype) = RMS norm of sum_s read[s] x_s, times w. */
+int b200_hyper_embed(const int32_t* tokens, const void* table, int dtype, float* x, int S, const float* read, const float* w, float eps,
+                     void* out, int T, int W, int vocab, void* stream);
+/* y = y1[t] (pitch ld1, or NULL) + sum_{c < nsum} y2_weight[t][c] y2[t nsum + c] (y2 or the weights may be NULL);
+ * x_d <- sum_s mix[s][d] x_s + write[d] y, every sum over the previous values (written back when store is set);
+ * out (out_dtype) = RMS norm of sum_d read[d] x_d of the NEW copies, times w: the next sublayer's input. */
+int b200_hyper_residual(float* x, int S, const float* y1, int ld1, const float* y2, int nsum, const float* y2_weight, const float* mix,
+                        const float* write, const float* read, const float* w, float eps, int store, void* out, int out_dtype, int T,
+                        int W, void* stream);
 
 #ifdef __cplusplus
 }

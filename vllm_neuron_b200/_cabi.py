@@ -12,7 +12,7 @@ _HERE = os.path.dirname(os.path.abspath(__file__))
 LIB_PATH = os.path.join(_HERE, "libb200_paged.so")
 
 OK = 0
-ABI_VERSION = 13
+ABI_VERSION = 14
 BF16, FP8_E4M3, INT8, F32 = 0, 1, 2, 3
 ACT_SWISH_CLAMPED, ACT_SILU, ACT_GELU_TANH = 0, 1, 2   # gate activation of a gated-linear unit
 ACT_NONE, ACT_RELU2 = 3, 4   # plain activation behind a bias: identity, square of relu
@@ -93,13 +93,14 @@ SIGNATURES = {
                                           _i, _i, _i, _p, _p, _p, _i, _i, _p]),
     "b200_attn_split_merge": (_i, [_p, _i, _i, _i, _i, _i, _p, _i64, _p]),
     "b200_qk_norm_rope_kv_write": (_i, [_p, _i, _i, _i, _i, _p, _p, _f, _i, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i,
-                                        _i, _i, _p, _i, _p]),
+                                        _i, _i, _p, _i, _p, _p]),
     "b200_moe_topk": (_i, [_p, _i, _p, _i, _p, _p, _i, _i, _i, _p]),
+    "b200_moe_topk_grouped": (_i, [_p, _i, _p, _i, _i, _f, _p, _p, _i, _i, _i, _p]),
     "b200_moe_tile_rows": (_i, []),
     "b200_moe_gather_scale": (_i, [_p, _i, _p, _i, _i, _p, _p, _i, _p, _i, _p]),
     "b200_moe_align": (_i, [_p, _i, _i, _p, _i, _p, _i, _p, _i, _p]),
     "b200_grouped_linear": (_i, [_p, _i, _p, _i, _p, _p, _i64, _p, _p, _i, _i, _i, _i, _i, _p, _i, _i, _i, _i, _f, _i, _p]),
-    "b200_batched_linear": (_i, [_p, _i, _i64, _p, _i64, _p, _i, _i64, _i, _i, _i, _i, _i, _i, _p, _i, _p]),
+    "b200_batched_linear": (_i, [_p, _i, _i64, _p, _i64, _p, _i, _i64, _i, _i, _i, _i, _i, _i, _p, _i, _i, _p]),
     # post-norm hybrid decoders: bigram embedding, RMS-norm residual steps, gated delta rule, latent attention
     "b200_embed_bigram": (_i, [_p, _p, _p, _i, _i, _i, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _f, _p]),
     "b200_rms_residual": (_i, [_p, _p, _i, _p, _p, _f, _f, _p, _i, _i, _i, _p]),
@@ -127,7 +128,10 @@ SIGNATURES = {
     "b200_delta_scan": (_i, [_p, _i, _p, _p, _p, _p, _p, _p, _p, _i, _i, _i, _i, _i, _i, _p]),
     "b200_latent_kv_write": (_i, [_p, _i, _i, _i, _i, _i, _p, _f, _p, _p, _p, _p, _p, _i, _i, _p]),
     "b200_latent_q_prep": (_i, [_p, _i, _i, _i, _i, _i, _i, _p, _p, _p, _p, _i, _p, _i, _p]),
-    "b200_latent_attn_decode": (_i, [_p, _i, _p, _p, _i64, _p, _p, _f, _p, _i, _i, _i, _i, _i, _p]),
+    "b200_latent_attn_decode": (_i, [_p, _i, _p, _p, _i64, _p, _p, _p, _f, _i, _p, _i, _i, _i, _i, _i, _p]),
+    # hyper-connections: several copies of the residual stream mixed around every sublayer
+    "b200_hyper_embed": (_i, [_p, _p, _i, _p, _i, _p, _p, _f, _p, _i, _i, _i, _p]),
+    "b200_hyper_residual": (_i, [_p, _i, _p, _i, _p, _i, _p, _p, _p, _p, _p, _f, _i, _p, _i, _i, _i, _p]),
 }
 
 _lib = None

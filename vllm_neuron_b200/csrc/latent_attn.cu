@@ -4,7 +4,7 @@
 //     score = (q' . c + q_rot . k_rot) * scale,      out_latent = sum_j p_j c_j,      value = W_uv out_latent,
 // which is multi-query attention with key rows [c | k_rot] (width C + R) and value rows c (the first C columns of the
 // same rows): the paged attention kernels of swa_attn.cu / swa_attn_prefill.cu serve it with one kv head, the value pool
-// aliased onto the key pool, no sink and no window.  This file holds the per-token steps around them:
+// aliased onto the key pool (a sliding window and a sink logit per head are options of those kernels and of the one here).  This file holds the per-token steps around them:
 //   * latent_kv_write: RMS norm of the latent (plain weight), rotation of the shared key part by the token's position
 //     (pairs (2i, 2i + 1) of the first rot_n columns; cos / sin come from a table [positions][rot_n / 2], so any frequency
 //     scaling lives in the table), scatter of the row into the pool by slot;
@@ -14,7 +14,8 @@
 //     the same cache rows, so the HEADS are the rows of the MMA tile: a CTA takes one token and up to 16 heads, its warps
 //     take the visible keys in tiles of 32 round-robin (each warp gathers its tile into its own shared-memory buffer with
 //     cp.async, S = Q K^T and O += P V on mma.sync m16n8k16 with the values read from the leading columns of the same
-//     tile, fp32 online softmax per warp) and merge through shared memory.
+//     tile, fp32 online softmax per warp) and merge through shared memory.  With a window the walk starts at its first key; a sink
+//     starts every warp's maximum and, in warp 0 alone, the denominator.
 #include <math.h>
 
 #include "hybrid_common.cuh"
@@ -94,8 +95,8 @@ template <int DV16M>  // accumulator capacity: Dv <= 16 * DV16M
 __global__ void __launch_bounds__(256)
     latent_attn_decode_kernel(const float* __restrict__ q, int ldq, const __nv_bfloat16* __restrict__ pool,
                               const int32_t* __restrict__ block_table, int64_t bt_stride, const int32_t* __restrict__ tok_row,
-                              const int32_t* __restrict__ tok_pos, float scale, __nv_bfloat16* __restrict__ out, int H, int D,
-                              int Dv, int bs) {
+                              const int32_t* __restrict__ tok_pos, const float* __restrict__ sink, float scale, int window,
+                              __nv_bfloat16* __restrict__ out, int H, int D, int Dv, int bs) {
   griddep_wait();
   extern __shared__ __align__(16) unsigned char la_sm[];
   const int nw = blockDim.x >> 5, warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -113,14 +114,18 @@ __global__ void __launch_bounds__(256)
     *reinterpret_cast<__nv_bfloat162*>(Qs + r * ldk + d) = __floats2bfloat162_rn(v.x, v.y);
   }
   __syncthreads();
-  float m_lo = -INFINITY, m_hi = -INFINITY, l_lo = 0.f, l_hi = 0.f;
+  const int r_lo = lane >> 2;
+  const int lo = pos - window + 1 > 0 ? pos - window + 1 : 0;  // the first visible key
+  float m_lo = sink && h0 + r_lo < H ? sink[h0 + r_lo] : -INFINITY, m_hi = sink && h0 + r_lo + 8 < H ? sink[h0 + r_lo + 8] : -INFINITY;
+  const bool count_sink = sink && warp == 0 && (lane & 3) == 0;  // the sink's 1 in the denominator, once per row
+  float l_lo = count_sink && h0 + r_lo < H ? 1.0f : 0.f, l_hi = count_sink && h0 + r_lo + 8 < H ? 1.0f : 0.f;
   float o[2 * DV16M][4];
 #pragma unroll
   for (int j = 0; j < 2 * DV16M; ++j)
 #pragma unroll
     for (int c = 0; c < 4; ++c) o[j][c] = 0.f;
   const int kch = D / 8;  // 16-byte chunks per cache row
-  for (int j0 = LD_KEYS * warp; j0 <= pos; j0 += LD_KEYS * nw) {
+  for (int j0 = lo + LD_KEYS * warp; j0 <= pos; j0 += LD_KEYS * nw) {
     // ---- this warp's 32 cache rows -> its buffer (rows past the token's position are zeros)
     const int jm = j0 + lane;
     const int64_t myrow = jm <= pos ? (int64_t)bt[jm / bs] * bs + (jm % bs) : -1;
@@ -213,7 +218,6 @@ __global__ void __launch_bounds__(256)
   l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 1);
   l_hi += __shfl_xor_sync(0xffffffffu, l_hi, 2);
   float* Os = reinterpret_cast<float*>(Kt);  // [16][Dv] fp32 fits: 32 rows of more than Dv bf16
-  const int r_lo = lane >> 2;
 #pragma unroll
   for (int j = 0; j < 2 * DV16M; ++j) {
     const int d = 8 * j + 2 * (lane & 3);
@@ -240,7 +244,7 @@ __global__ void __launch_bounds__(256)
     for (int w = 0; w < nw; ++w) mt = fmaxf(mt, ml[(w * 16 + r) * 2]);
     float lt = 0.f, v = 0.f;
     for (int w = 0; w < nw; ++w) {
-      const float f = __expf(ml[(w * 16 + r) * 2] - mt);  // a warp without keys holds m = -inf, l = 0, O = 0
+      const float f = __expf(ml[(w * 16 + r) * 2] - mt);  // a warp without keys holds O = 0, m = -inf or the sink, l = 0 (1: the sink)
       lt += ml[(w * 16 + r) * 2 + 1] * f;
       v += O0[w * wstride + r * Dv + d] * f;
     }
@@ -280,9 +284,10 @@ int b200_latent_q_prep(const float* q, int ldq, int H, int D, int R, int rot_n, 
 }
 
 int b200_latent_attn_decode(const float* q, int ldq, const void* pool, const int32_t* block_table, int64_t bt_stride,
-                            const int32_t* tok_row, const int32_t* tok_pos, float scale, void* out, int T, int H, int D, int Dv,
-                            int block_size, void* stream) {
+                            const int32_t* tok_row, const int32_t* tok_pos, const float* sink, float scale, int window, void* out,
+                            int T, int H, int D, int Dv, int block_size, void* stream) {
   B200_REQUIRE(q && pool && block_table && tok_row && tok_pos && out, "latent_attn_decode: null pointer");
+  B200_REQUIRE(window >= 1, "latent_attn_decode: window %d", window);
   if (D % 16 || Dv % 16 || Dv > 256 || Dv > D || D > 1024 || (ldq & 1) || ((uintptr_t)q & 7) || H < 1) {
     set_last_error("latent_attn_decode: row width %d / value width %d need multiples of 16 (values <= 256)", D, Dv);
     return B200_ERR_UNSUPPORTED;
@@ -299,8 +304,8 @@ int b200_latent_attn_decode(const float* q, int ldq, const void* pool, const int
     if (smem > 48 * 1024)                                                                                                      \
       B200_CUDA_OK(cudaFuncSetAttribute(latent_attn_decode_kernel<M>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
     B200_CUDA_OK(launch_kernel(latent_attn_decode_kernel<M>, grid, dim3(nw * 32), smem, (cudaStream_t)stream, q, ldq,          \
-                               (const BT*)pool, block_table, bt_stride, tok_row, tok_pos, scale, (BT*)out, H, D, Dv,          \
-                               block_size));                                                                                   \
+                               (const BT*)pool, block_table, bt_stride, tok_row, tok_pos, sink, scale, window, (BT*)out, H, D, \
+                               Dv, block_size));                                                                               \
   } while (0)
   if (Dv <= 64) LAD_LAUNCH(4);
   else if (Dv <= 128) LAD_LAUNCH(8);

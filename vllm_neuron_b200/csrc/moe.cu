@@ -2,6 +2,8 @@
 //   * moe_topk: over the fp32 router logits (a linear of the layer's input, plus an optional per-expert bias): the `top`
 //     largest are chosen (ties go to the lower expert index); the routing weights are either the sigmoid of each chosen
 //     logit (no renormalisation) or the softmax over the chosen logits only;
+//   * moe_topk_grouped: softmax scores over all experts, the choice made on score + correction among the experts of the best
+//     groups of neighbours, the scores themselves (times a constant) as weights;
 //   * moe_align: counting sort of the (token, choice) pairs by expert into row tiles of MOE_BM, each tile owned by one
 //     expert (ragged tails padded with -1), so the expert GEMMs run as one launch without the host knowing the counts;
 //   * grouped_linear: out = A W_e^T with fp32 accumulation over K in ascending order (the result of a row does not depend
@@ -67,6 +69,79 @@ __global__ void moe_topk_kernel(const float* __restrict__ z, int ld, const float
   }
 }
 
+// One warp per token.  s = softmax(z) over all E experts (fp32), choice = s + correction.  The experts form `groups` equal runs of
+// neighbours; a run's rank is its largest choice score, and only the best `keep` runs stay eligible (the rest is masked with -inf: a
+// correction may push eligible scores below zero).  The `top` largest choice scores win (ties to the lower index);
+// weight = s (without the correction) * scale, not renormalised.
+__global__ void moe_topk_grouped_kernel(const float* __restrict__ z, int ld, const float* __restrict__ correction, int E, int groups,
+                                        int keep, int top, float scale, int32_t* __restrict__ idx, float* __restrict__ wt, int ntok) {
+  griddep_launch();
+  griddep_wait();
+  extern __shared__ float tg_sm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+  const int t = blockIdx.x * nw + warp;
+  if (t >= ntok) return;
+  float* s = tg_sm + warp * (2 * E + groups);  // [E] scores
+  float* ch = s + E;                           // [E] choice scores; -inf: taken or out
+  float* gb = ch + E;                          // [groups] best choice score; -inf: kept already
+  const float* zr = z + (int64_t)t * ld;
+  const int gs = E / groups;
+  float m = -INFINITY, sum = 0.f;
+  for (int e = lane; e < E; e += 32) m = fmaxf(m, zr[e]);
+  m = warp_max(m);
+  for (int e = lane; e < E; e += 32) {
+    s[e] = expf(zr[e] - m);
+    sum += s[e];
+  }
+  sum = warp_sum(sum);
+  for (int e = lane; e < E; e += 32) {
+    s[e] = s[e] / sum;
+    ch[e] = s[e] + (correction ? correction[e] : 0.f);
+  }
+  __syncwarp();
+  // the position of the largest of v[0 .. n) (lowest index among equals; 0 when nothing is above -inf)
+  auto best_of = [&](const float* v, int n) -> int {
+    float b = -INFINITY;
+    int bi = n;
+    for (int i = lane; i < n; i += 32)
+      if (v[i] > b) b = v[i], bi = i;
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, b, o);
+      const int oi = __shfl_xor_sync(0xffffffffu, bi, o);
+      if (ob > b || (ob == b && oi < bi)) b = ob, bi = oi;
+    }
+    return bi < n ? bi : 0;
+  };
+  if (groups > 1 && keep < groups) {
+    for (int g = lane; g < groups; g += 32) {
+      float b = -INFINITY;
+      for (int i = 0; i < gs; ++i) b = fmaxf(b, ch[g * gs + i]);
+      gb[g] = b;
+    }
+    __syncwarp();
+    for (int k = 0; k < keep; ++k) {
+      const int g = best_of(gb, groups);
+      __syncwarp();
+      if (lane == 0) gb[g] = -INFINITY;
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (gb[e / gs] != -INFINITY) ch[e] = -INFINITY;
+    __syncwarp();
+  }
+  for (int c = 0; c < top; ++c) {
+    const int e = best_of(ch, E);
+    __syncwarp();
+    if (lane == 0) {
+      idx[(int64_t)t * top + c] = e;
+      wt[(int64_t)t * top + c] = s[e] * scale;
+      ch[e] = -INFINITY;
+    }
+    __syncwarp();
+  }
+}
+
 // single CTA: counts -> padded offsets -> tile owners -> scatter of pair ids
 __global__ void moe_align_kernel(const int32_t* __restrict__ idx, int npairs, int E, int32_t* __restrict__ sorted_ids, int cap,
                                  int32_t* __restrict__ tile_expert, int max_tiles, int32_t* __restrict__ num_tiles, int bm) {
@@ -117,7 +192,7 @@ __global__ void __launch_bounds__(GL_THREADS)
                           const float* __restrict__ row_scale, const T* __restrict__ w, int64_t w_stride,
                           const int32_t* __restrict__ tile_expert, const int32_t* __restrict__ num_tiles, int M, int N, int K,
                           void* __restrict__ out, int ldo, int scatter, float limit, int act, int64_t a_zs, int64_t o_zs,
-                          int store_typed, const float* __restrict__ gate, int gate_ld) {
+                          int store_typed, const float* __restrict__ gate, int gate_ld, int gate_cols) {
   griddep_launch();
   griddep_wait();
   constexpr int NW = EPI == GL_EPI_GLU ? 2 : 1;
@@ -201,7 +276,7 @@ __global__ void __launch_bounds__(GL_THREADS)
         stf((T*)out, o, glu_act(acc[0][i][j], acc[NW - 1][i][j], act, limit));
       } else {
         float v = acc[0][i][j];
-        if (gate) v *= 1.0f / (1.0f + expf(-gate[(int64_t)dst * gate_ld + blockIdx.z]));
+        if (gate) v *= 1.0f / (1.0f + expf(-gate[(int64_t)dst * gate_ld + (gate_cols ? blockIdx.z * N + n : blockIdx.z)]));
         if (store_typed) stf((T*)out, o, v);
         else ((float*)out)[o] = v;
       }
@@ -224,7 +299,7 @@ __global__ void __launch_bounds__(128)
                        const float* __restrict__ row_scale, const __nv_bfloat16* __restrict__ w, int64_t w_stride,
                        const int32_t* __restrict__ tile_expert, const int32_t* __restrict__ num_tiles, int M, int N, int K,
                        void* __restrict__ out, int ldo, int scatter, float limit, int act, int64_t a_zs, int64_t o_zs,
-                       int store_typed, const float* __restrict__ gate, int gate_ld) {
+                       int store_typed, const float* __restrict__ gate, int gate_ld, int gate_cols) {
   griddep_launch();
   griddep_wait();
   constexpr int R = 1;            // 32-row sub-tiles per CTA (prompt-sized batches take grouped_mma_pipe_kernel instead)
@@ -361,12 +436,13 @@ __global__ void __launch_bounds__(128)
               __float2bfloat16_rn(glu_act(acc[mt][j][c], acc[mt][j + 2][c], act, limit));
         }
       } else {
-        const float gt = gate ? 1.0f / (1.0f + expf(-gate[(int64_t)dst * gate_ld + blockIdx.z])) : 1.0f;
+        float gt = gate && !gate_cols ? 1.0f / (1.0f + expf(-gate[(int64_t)dst * gate_ld + blockIdx.z])) : 1.0f;
 #pragma unroll
         for (int j = 0; j < 4; ++j) {
           const int n = n0 + 32 * warp + 8 * j + col;
           if (n >= N) continue;
           const int64_t o = (int64_t)blockIdx.z * o_zs + (int64_t)dst * ldo + n;
+          if (gate_cols) gt = 1.0f / (1.0f + expf(-gate[(int64_t)dst * gate_ld + blockIdx.z * N + n]));
           if (store_typed) ((__nv_bfloat16*)out)[o] = __float2bfloat16_rn(acc[mt][j][c] * gt);
           else ((float*)out)[o] = acc[mt][j][c] * gt;
         }
@@ -556,6 +632,20 @@ int b200_moe_topk(const float* logits, int ld, const float* bias, int mode, int3
   return B200_OK;
 }
 
+int b200_moe_topk_grouped(const float* logits, int ld, const float* correction, int groups, int keep, float scale, int32_t* topk_idx,
+                          float* topk_weight, int T, int E, int top, void* stream) {
+  B200_REQUIRE(logits && topk_idx && topk_weight, "moe_topk_grouped: null pointer");
+  B200_REQUIRE(E >= 1 && E <= 4096 && ld >= E && groups >= 1 && E % groups == 0 && keep >= 1 && keep <= groups,
+               "moe_topk_grouped: %d experts in %d groups of which %d are kept", E, groups, keep);
+  B200_REQUIRE(top >= 1 && top <= keep * (E / groups), "moe_topk_grouped: top %d of %d experts in reach", top, keep * (E / groups));
+  if (T <= 0) return B200_OK;
+  const size_t per = (size_t)(2 * E + groups) * 4;  // at most 48 KB for one warp
+  const int warps = per * 4 <= 48 * 1024 ? 4 : per * 2 <= 48 * 1024 ? 2 : 1;
+  B200_CUDA_OK(launch_kernel(moe_topk_grouped_kernel, dim3((T + warps - 1) / warps), dim3(32 * warps), per * warps,
+                             (cudaStream_t)stream, logits, ld, correction, E, groups, keep, top, scale, topk_idx, topk_weight, T));
+  return B200_OK;
+}
+
 int b200_moe_tile_rows(void) { return MOE_BM; }
 
 int b200_moe_gather_scale(const void* h, int ldh, const int32_t* sorted_ids, int cap, int top, const float* weight,
@@ -603,7 +693,7 @@ int b200_grouped_linear(const void* a, int lda, const int32_t* sorted_ids, int g
 #define GM_LAUNCH(EPI, BN)                                                                                                   \
   B200_CUDA_OK(launch_kernel(grouped_mma_kernel<EPI>, dim3(row_tiles, (N + BN - 1) / BN), dim3(128), 0, st, (const BT*)a, lda, \
                              sorted_ids, gather_div, row_scale, (const BT*)w, w_expert_stride, tile_expert, num_tiles, M, N, K, \
-                             out, ldo, scatter, limit, act, (int64_t)0, (int64_t)0, 0, no_gate, 0))
+                             out, ldo, scatter, limit, act, (int64_t)0, (int64_t)0, 0, no_gate, 0, 0))
     if (tile_rows == MOE_BM) {
       if (glu) GM_LAUNCH(GL_EPI_GLU, 64);
       else GM_LAUNCH(GL_EPI_STORE, 128);
@@ -631,20 +721,20 @@ int b200_grouped_linear(const void* a, int lda, const int32_t* sorted_ids, int g
     if (glu)
       B200_CUDA_OK(launch_kernel(grouped_linear_kernel<ET, GL_EPI_GLU>, grid, dim3(GL_THREADS), 0, st, (const ET*)a, lda, sorted_ids,
                                  gather_div, row_scale, (const ET*)w, w_expert_stride, tile_expert, num_tiles, M, N, K, out, ldo,
-                                 scatter, limit, act, (int64_t)0, (int64_t)0, 0, no_gate, 0));
+                                 scatter, limit, act, (int64_t)0, (int64_t)0, 0, no_gate, 0, 0));
     else
       B200_CUDA_OK(launch_kernel(grouped_linear_kernel<ET, GL_EPI_STORE>, grid, dim3(GL_THREADS), 0, st, (const ET*)a, lda,
                                  sorted_ids, gather_div, row_scale, (const ET*)w, w_expert_stride, tile_expert, num_tiles, M, N, K,
-                                 out, ldo, scatter, limit, act, (int64_t)0, (int64_t)0, 0, no_gate, 0));
+                                 out, ldo, scatter, limit, act, (int64_t)0, (int64_t)0, 0, no_gate, 0, 0));
   });
   return B200_OK;
 }
 
 int b200_batched_linear(const void* a, int lda, int64_t a_batch_stride, const void* w, int64_t w_batch_stride, void* out, int ldo,
                         int64_t out_batch_stride, int batch, int M, int N, int K, int dtype, int out_typed, const float* gate,
-                        int gate_ld, void* stream) {
+                        int gate_ld, int gate_cols, void* stream) {
   B200_REQUIRE(a && w && out, "batched_linear: null pointer");
-  B200_REQUIRE(N > 0 && K > 0 && batch >= 1 && batch <= 65535, "batched_linear: bad shape N=%d K=%d batch=%d", N, K, batch);
+  B200_REQUIRE(N > 0 && K > 0 && batch >= 1 && batch <= 65535 && (gate || !gate_cols), "batched_linear: bad shape N=%d K=%d batch=%d", N, K, batch);
   if (M <= 0) return B200_OK;
   cudaStream_t st = (cudaStream_t)stream;
   const int row_tiles = (M + MOE_BM - 1) / MOE_BM;
@@ -656,14 +746,14 @@ int b200_batched_linear(const void* a, int lda, int64_t a_batch_stride, const vo
     using BT = __nv_bfloat16;
     B200_CUDA_OK(launch_kernel(grouped_mma_kernel<GL_EPI_STORE>, dim3(row_tiles, (N + 127) / 128, batch), dim3(128), 0, st,
                                (const BT*)a, lda, none, 0, no_scale, (const BT*)w, w_batch_stride, none, none, M, N, K, out, ldo, 0,
-                               0.f, 0, a_batch_stride, out_batch_stride, out_typed, gate, gate_ld));
+                               0.f, 0, a_batch_stride, out_batch_stride, out_typed, gate, gate_ld, gate_cols));
     return B200_OK;
   }
   dim3 grid(row_tiles, (N + GL_BN - 1) / GL_BN, batch);
   B200_DISPATCH_ELEM(dtype, ET,
                      B200_CUDA_OK(launch_kernel(grouped_linear_kernel<ET, GL_EPI_STORE>, grid, dim3(GL_THREADS), 0, st, (const ET*)a,
                                                 lda, none, 0, no_scale, (const ET*)w, w_batch_stride, none, none, M, N, K, out, ldo, 0,
-                                                0.f, 0, a_batch_stride, out_batch_stride, out_typed, gate, gate_ld)));
+                                                0.f, 0, a_batch_stride, out_batch_stride, out_typed, gate, gate_ld, gate_cols)));
   return B200_OK;
 }
 

@@ -50,13 +50,17 @@ __global__ void kv_write_vmix_kernel(const float* __restrict__ qkv, int ld, int 
 
 // 1 / rms of every q head (inv[0 .. H)) and k head (inv[H .. H + G)), a warp per head; a side without a norm is left out
 __device__ __forceinline__ void head_inverse_rms(const float* row, int q_col0, int k_col0, bool q_norm, bool k_norm, int H, int G,
-                                                 int D, float eps, float* inv) {
+                                                 int D, float eps, float* inv, const float* q_bias, const float* k_bias) {
   const int lane = threadIdx.x & 31;
   for (int i = threadIdx.x >> 5; i < H + G; i += blockDim.x >> 5) {
     if (!(i < H ? q_norm : k_norm)) continue;
     const float* r = row + (i < H ? q_col0 + i * D : k_col0 + (i - H) * D);
+    const float* bias = i < H ? (q_bias ? q_bias + i * D : nullptr) : (k_bias ? k_bias + (i - H) * D : nullptr);
     float ss = 0.f;
-    for (int d = lane; d < D; d += 32) ss += r[d] * r[d];
+    for (int d = lane; d < D; d += 32) {
+      const float v = r[d] + (bias ? bias[d] : 0.f);
+      ss += v * v;
+    }
     ss = warp_sum(ss);
     if (lane == 0) inv[i] = 1.0f / sqrtf(ss / (float)D + eps);
   }
@@ -67,7 +71,8 @@ __device__ __forceinline__ void head_inverse_rms(const float* row, int q_col0, i
 // multiplied by a weight per column -- or, with head_norm, each head by its own RMS and a weight [D] that the heads share --, then the first rot_n
 // columns of every head turn by the token's position: column pairs (i, i + rot_n / 2) when rot_half, else (2i, 2i + 1); a pair
 // (u, v) becomes (u cos - v sin, v cos + u sin) with cos / sin from fp32 tables [positions][rot_n / 2] (any frequency
-// scaling and magnitude factor live in the tables).  q goes to q_out fp32 [T][H * D]; k and v to the pools by slot.
+// scaling and magnitude factor live in the tables).  bias (or NULL) fp32 [q: H * D | k: G * D | v: Gv * Dv]: the projections' biases,
+// added first.  q goes to q_out fp32 [T][H * D]; k and v to the pools by slot.
 template <typename KT>
 __global__ void qk_norm_rope_kv_write_kernel(const float* __restrict__ src, int ld, int q_col0, int k_col0, int v_col0,
                                              const float* __restrict__ q_norm, const float* __restrict__ k_norm, float eps,
@@ -75,7 +80,7 @@ __global__ void qk_norm_rope_kv_write_kernel(const float* __restrict__ src, int 
                                              const float* __restrict__ sin_t, const int32_t* __restrict__ tok_pos,
                                              const int64_t* __restrict__ slots, float* __restrict__ q_out, KT* __restrict__ k_pool,
                                              KT* __restrict__ v_pool, int H, int G, int Gv, int D, int Dv, int bs,
-                                             const float* __restrict__ q_head_scale, int head_norm) {
+                                             const float* __restrict__ q_head_scale, int head_norm, const float* __restrict__ bias) {
   griddep_launch();
   griddep_wait();
   extern __shared__ float inv_h[];  // head_norm: [H + G]
@@ -83,16 +88,23 @@ __global__ void qk_norm_rope_kv_write_kernel(const float* __restrict__ src, int 
   const int t = blockIdx.x;
   const float* row = src + (int64_t)t * ld;
   const int nq = H * D, nk = G * D;
+  const float *qb = bias, *kb = bias ? bias + nq : nullptr, *vb = bias ? bias + nq + nk : nullptr;
   float inv_q = 1.0f, inv_k = 1.0f;
   if (head_norm) {
-    head_inverse_rms(row, q_col0, k_col0, q_norm != nullptr, k_norm != nullptr, H, G, D, eps, inv_h);
+    head_inverse_rms(row, q_col0, k_col0, q_norm != nullptr, k_norm != nullptr, H, G, D, eps, inv_h, qb, kb);
     __syncthreads();
   } else if (q_norm || k_norm) {  // sums of squares over the whole projections
     float sq = 0.f, sk = 0.f;
     if (q_norm)
-      for (int i = threadIdx.x; i < nq; i += blockDim.x) sq += row[q_col0 + i] * row[q_col0 + i];
+      for (int i = threadIdx.x; i < nq; i += blockDim.x) {
+        const float u = row[q_col0 + i] + (qb ? qb[i] : 0.f);
+        sq += u * u;
+      }
     if (k_norm)
-      for (int i = threadIdx.x; i < nk; i += blockDim.x) sk += row[k_col0 + i] * row[k_col0 + i];
+      for (int i = threadIdx.x; i < nk; i += blockDim.x) {
+        const float u = row[k_col0 + i] + (kb ? kb[i] : 0.f);
+        sk += u * u;
+      }
     sq = warp_sum(sq);
     sk = warp_sum(sk);
     if ((threadIdx.x & 31) == 0) {
@@ -121,13 +133,13 @@ __global__ void qk_norm_rope_kv_write_kernel(const float* __restrict__ src, int 
   const int64_t slot = slots[t];
   const int64_t blk = slot / bs, off = slot % bs;
   // the value of column i of a projection after its norm
-  auto turned = [&](int col0, const float* nw, float inv, int i) -> float {
+  auto turned = [&](int col0, const float* nw, float inv, const float* b, int i) -> float {
     const int d = i % D;
     if (head_norm && nw) {
       inv = inv_h[(col0 == q_col0 ? 0 : H) + i / D];
       nw -= i - d;  // the weight is per column of a head
     }
-    const float u = row[col0 + i] * (nw ? inv * nw[i] : 1.0f);
+    const float u = (row[col0 + i] + (b ? b[i] : 0.f)) * (nw ? inv * nw[i] : 1.0f);
     if (d >= rot_n) return u;
     int partner, idx;
     bool first;
@@ -138,21 +150,21 @@ __global__ void qk_norm_rope_kv_write_kernel(const float* __restrict__ src, int 
     } else {
       first = (d & 1) == 0;
       idx = d >> 1;
-      partner = i ^ 1;
+      partner = first ? i + 1 : i - 1;
     }
-    const float o = row[col0 + partner] * (nw ? inv * nw[partner] : 1.0f);
+    const float o = (row[col0 + partner] + (b ? b[partner] : 0.f)) * (nw ? inv * nw[partner] : 1.0f);
     return first ? u * cs[idx] - o * sn[idx] : u * cs[idx] + o * sn[idx];
   };
   for (int i = threadIdx.x; i < nq; i += blockDim.x)
-    q_out[(int64_t)t * nq + i] = turned(q_col0, q_norm, inv_q, i) * (q_head_scale ? q_head_scale[i / D] : 1.0f);
+    q_out[(int64_t)t * nq + i] = turned(q_col0, q_norm, inv_q, qb, i) * (q_head_scale ? q_head_scale[i / D] : 1.0f);
   if (slot < 0) return;
   for (int i = threadIdx.x; i < nk; i += blockDim.x) {
     const int g = i / D, d = i - g * D;
-    stf(k_pool, ((blk * G + g) * bs + off) * D + d, turned(k_col0, k_norm, inv_k, i));
+    stf(k_pool, ((blk * G + g) * bs + off) * D + d, turned(k_col0, k_norm, inv_k, kb, i));
   }
   for (int i = threadIdx.x; i < Gv * Dv; i += blockDim.x) {
     const int g = i / Dv, d = i - g * Dv;
-    stf(v_pool, ((blk * Gv + g) * bs + off) * Dv + d, row[v_col0 + i]);
+    stf(v_pool, ((blk * Gv + g) * bs + off) * Dv + d, row[v_col0 + i] + (vb ? vb[i] : 0.f));
   }
 }
 
@@ -166,7 +178,7 @@ __global__ void qk_norm_rope_kv_write_vec_kernel(const float* __restrict__ src, 
                                                  const float* __restrict__ sin_t, const int32_t* __restrict__ tok_pos,
                                                  const int64_t* __restrict__ slots, float* __restrict__ q_out,
                                                  KT* __restrict__ k_pool, KT* __restrict__ v_pool, int H, int G, int Gv, int D, int Dv,
-                                                 int bs, const float* __restrict__ q_head_scale, int head_norm) {
+                                                 int bs, const float* __restrict__ q_head_scale, int head_norm, const float* __restrict__ bias) {
   griddep_launch();
   griddep_wait();
   extern __shared__ float inv_h[];  // head_norm: [H + G]
@@ -174,21 +186,31 @@ __global__ void qk_norm_rope_kv_write_vec_kernel(const float* __restrict__ src, 
   const int t = blockIdx.x;
   const float* row = src + (int64_t)t * ld;
   const int nq = H * D, nk = G * D;
+  const float *qb = bias, *kb = bias ? bias + nq : nullptr, *vb = bias ? bias + nq + nk : nullptr;
   auto ld4 = [](const float* p) { return *reinterpret_cast<const float4*>(p); };
+  // four columns of a projection with its bias
+  auto raw4 = [&](int col0, const float* b, int i) -> float4 {
+    float4 u = ld4(row + col0 + i);
+    if (b) {
+      const float4 v = ld4(b + i);
+      u.x += v.x, u.y += v.y, u.z += v.z, u.w += v.w;
+    }
+    return u;
+  };
   float inv_q = 1.0f, inv_k = 1.0f;
   if (head_norm) {
-    head_inverse_rms(row, q_col0, k_col0, q_norm != nullptr, k_norm != nullptr, H, G, D, eps, inv_h);
+    head_inverse_rms(row, q_col0, k_col0, q_norm != nullptr, k_norm != nullptr, H, G, D, eps, inv_h, qb, kb);
     __syncthreads();
   } else if (q_norm || k_norm) {
     float sq = 0.f, sk = 0.f;
     if (q_norm)
       for (int i = threadIdx.x * 4; i < nq; i += blockDim.x * 4) {
-        const float4 a = ld4(row + q_col0 + i);
+        const float4 a = raw4(q_col0, qb, i);
         sq += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
       }
     if (k_norm)
       for (int i = threadIdx.x * 4; i < nk; i += blockDim.x * 4) {
-        const float4 a = ld4(row + k_col0 + i);
+        const float4 a = raw4(k_col0, kb, i);
         sk += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
       }
     sq = warp_sum(sq);
@@ -219,8 +241,8 @@ __global__ void qk_norm_rope_kv_write_vec_kernel(const float* __restrict__ src, 
   const int64_t slot = slots[t];
   const int64_t blk = slot / bs, off = slot % bs;
   // columns i .. i + 3 of a projection after norm and rotation; d = i % D
-  auto normed = [&](int col0, const float* nw, float inv, int i) -> float4 {
-    float4 u = ld4(row + col0 + i);
+  auto normed = [&](int col0, const float* nw, float inv, const float* b, int i) -> float4 {
+    float4 u = raw4(col0, b, i);
     if (nw) {
       if (head_norm) {
         const int hd = i / D;
@@ -232,13 +254,13 @@ __global__ void qk_norm_rope_kv_write_vec_kernel(const float* __restrict__ src, 
     }
     return u;
   };
-  auto turned = [&](int col0, const float* nw, float inv, int i, int d) -> float4 {
-    const float4 u = normed(col0, nw, inv, i);
+  auto turned = [&](int col0, const float* nw, float inv, const float* b, int i, int d) -> float4 {
+    const float4 u = normed(col0, nw, inv, b, i);
     if (d >= rot_n) return u;
     if (rot_half) {
       const bool first = d < half;
       const int idx = first ? d : d - half;
-      const float4 o = normed(col0, nw, inv, first ? i + half : i - half);
+      const float4 o = normed(col0, nw, inv, b, first ? i + half : i - half);
       const float4 c = ld4(cs + idx), s = ld4(sn + idx);
       if (first) return make_float4(u.x * c.x - o.x * s.x, u.y * c.y - o.y * s.y, u.z * c.z - o.z * s.z, u.w * c.w - o.w * s.w);
       return make_float4(u.x * c.x + o.x * s.x, u.y * c.y + o.y * s.y, u.z * c.z + o.z * s.z, u.w * c.w + o.w * s.w);
@@ -255,7 +277,7 @@ __global__ void qk_norm_rope_kv_write_vec_kernel(const float* __restrict__ src, 
     }
   };
   for (int i = threadIdx.x * 4; i < nq; i += blockDim.x * 4) {
-    float4 r = turned(q_col0, q_norm, inv_q, i, i % D);
+    float4 r = turned(q_col0, q_norm, inv_q, qb, i, i % D);
     if (q_head_scale) {  // D % 4 == 0: the four columns belong to one head
       const float hs = q_head_scale[i / D];
       r.x *= hs, r.y *= hs, r.z *= hs, r.w *= hs;
@@ -265,11 +287,11 @@ __global__ void qk_norm_rope_kv_write_vec_kernel(const float* __restrict__ src, 
   if (slot < 0) return;
   for (int i = threadIdx.x * 4; i < nk; i += blockDim.x * 4) {
     const int g = i / D, d = i - g * D;
-    put(k_pool + ((blk * G + g) * bs + off) * D + d, turned(k_col0, k_norm, inv_k, i, d));
+    put(k_pool + ((blk * G + g) * bs + off) * D + d, turned(k_col0, k_norm, inv_k, kb, i, d));
   }
   for (int i = threadIdx.x * 4; i < Gv * Dv; i += blockDim.x * 4) {
     const int g = i / Dv, d = i - g * Dv;
-    put(v_pool + ((blk * Gv + g) * bs + off) * Dv + d, ld4(row + v_col0 + i));
+    put(v_pool + ((blk * Gv + g) * bs + off) * Dv + d, raw4(v_col0, vb, i));
   }
 }
 
@@ -652,9 +674,10 @@ int b200_qk_norm_rope_kv_write(const float* src, int ld, int q_col0, int k_col0,
                                const float* k_norm, float eps, int rot_n, int rot_half, const float* cos_table,
                                const float* sin_table, const int32_t* tok_pos, const int64_t* slot_mapping, float* q_out,
                                void* k_pool, void* v_pool, int kv_dtype, int T, int H, int G, int Gv, int D, int Dv, int block_size,
-                               const float* q_head_scale, int head_norm, void* stream) {
+                               const float* q_head_scale, int head_norm, const float* bias, void* stream) {
   B200_REQUIRE(H + G <= 12000, "qk_norm_rope_kv_write: %d heads", H + G);
   B200_REQUIRE(!head_norm || q_col0 != k_col0, "qk_norm_rope_kv_write: q and k share their columns");
+  B200_REQUIRE(!bias || k_col0 != v_col0, "qk_norm_rope_kv_write: values that are the keys have no bias of their own");
   B200_REQUIRE(src && tok_pos && slot_mapping && q_out && k_pool && v_pool, "qk_norm_rope_kv_write: null pointer");
   B200_REQUIRE(rot_n >= 0 && rot_n <= D && rot_n % 2 == 0 && (rot_n == 0 || (cos_table && sin_table)),
                "qk_norm_rope_kv_write: %d rotating columns in heads of %d", rot_n, D);
@@ -664,7 +687,7 @@ int b200_qk_norm_rope_kv_write(const float* src, int ld, int q_col0, int k_col0,
   auto a16 = [](const void* p) { return ((uintptr_t)p & 15) == 0; };
   const bool vec = D % 4 == 0 && Dv % 4 == 0 && ld % 4 == 0 && q_col0 % 4 == 0 && k_col0 % 4 == 0 && v_col0 % 4 == 0 &&
                    rot_n % (rot_half ? 8 : 4) == 0 && a16(src) && a16(q_out) && a16(k_pool) && a16(v_pool) && a16(q_norm) &&
-                   a16(k_norm) && a16(cos_table) && a16(sin_table);
+                   a16(k_norm) && a16(bias) && a16(cos_table) && a16(sin_table);
   if (vec) {
     const int cols = H * D > G * D ? H * D : G * D;
     const int threads = cols >= 1024 ? 256 : cols >= 512 ? 128 : 64;
@@ -672,14 +695,14 @@ int b200_qk_norm_rope_kv_write(const float* src, int ld, int q_col0, int k_col0,
                        B200_CUDA_OK(launch_kernel(qk_norm_rope_kv_write_vec_kernel<KT>, dim3(T), dim3(threads), smem, (cudaStream_t)stream,
                                                   src, ld, q_col0, k_col0, v_col0, q_norm, k_norm, eps, rot_n, rot_half, cos_table,
                                                   sin_table, tok_pos, slot_mapping, q_out, (KT*)k_pool, (KT*)v_pool, H, G, Gv, D, Dv,
-                                                  block_size, q_head_scale, head_norm)));
+                                                  block_size, q_head_scale, head_norm, bias)));
     return B200_OK;
   }
   B200_DISPATCH_ELEM(kv_dtype, KT,
                      B200_CUDA_OK(launch_kernel(qk_norm_rope_kv_write_kernel<KT>, dim3(T), dim3(256), smem, (cudaStream_t)stream, src, ld,
                                                 q_col0, k_col0, v_col0, q_norm, k_norm, eps, rot_n, rot_half, cos_table, sin_table,
                                                 tok_pos, slot_mapping, q_out, (KT*)k_pool, (KT*)v_pool, H, G, Gv, D, Dv, block_size,
-                                                q_head_scale, head_norm)));
+                                                q_head_scale, head_norm, bias)));
   return B200_OK;
 }
 

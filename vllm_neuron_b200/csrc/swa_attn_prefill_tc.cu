@@ -472,7 +472,7 @@ extern "C" {
 // 1 when b200_swa_sink_attn_prefill_tc has a kernel for these head sizes and variants
 int b200_swa_sink_attn_prefill_tc_supported(int D, int Dv, int block_size, int v_div, int capped, int sigmoid) {
   if (block_size != TP_BLK || (capped && sigmoid)) return 0;
-  if (v_div == 1) return (D == 64 && Dv == 64) || (D == 128 && Dv == 128);
+  if (v_div == 1) return (D == 64 && Dv == 64) || (D == 128 && Dv == 128) || (D == 128 && Dv == 64 && !sigmoid);
   if (v_div == 2) return !capped && !sigmoid && (D == 32 || D == 64) && (Dv == 64 || Dv == 128);
   return 0;
 }
@@ -518,6 +518,10 @@ int b200_swa_sink_attn_prefill_tc(const float* q, int ldq, const void* k_pool, c
     if (sigmoid_bias) TP_GO(64, 64, TP_SIGMOID, false);
     if (softcap > 0.f) TP_GO(64, 64, TP_CAPPED, false);
     TP_GO(64, 64, TP_SOFTMAX, false);
+  }
+  if (Dv == 64) {
+    if (softcap > 0.f) TP_GO(128, 64, TP_CAPPED, false);
+    TP_GO(128, 64, TP_SOFTMAX, false);
   }
   if (sigmoid_bias) TP_GO(128, 128, TP_SIGMOID, false);
   if (softcap > 0.f) TP_GO(128, 128, TP_CAPPED, false);

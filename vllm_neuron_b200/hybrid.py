@@ -73,6 +73,17 @@ sublayers read x itself.  Mixers:
              per-head RMS norm, a sigmoid output gate.  State per sequence: S, the normaliser and the maximum (fp32).
 Feed-forward: W_down relu(W_up h)^2 with biases, or none.
 
+A sixth block style, pre-norm sublayers inside hyper-connections (the "Natalorn" design):
+  the residual stream is `streams` copies x_s;  u = sum_s r_s x_s;  y = sublayer(N(u));  x_t <- sum_s M[s, t] x_s + o_t y  with N a
+  plain RMS norm and r, M, o per sublayer; the logits read the norm of the copies' sum.  A run of layers may repeat as above, every
+  repetition with pools of its own.  Mixers:
+  * 'attention'        -- `RotAttnSpec` without rotation: sliding window, softmax;
+  * 'attention_2'      -- the same with projection biases, soft-capped scores and keys confined to the query's chunk;
+  * 'latent_attention' -- `LatentAttnSpec` with a sliding window, a sink logit per head and an elementwise sigmoid gate on the
+                          concatenated heads.
+Feed-forward: SiLU experts, softmax scores over all experts, chosen by score + correction among the experts of the best groups
+of neighbours, weighed on their outputs by score * router.scale; plus an always-on shared expert.
+
 The step is ONE ragged batch (`StepMeta`): portions of prompts and single decoded tokens run through the same kernels, each
 sequence continuing from its KV pages (block table row) and its state slot.  fp32 everywhere the design asks for it
 (residual stream, norms, softmax, router, recurrence); GEMM operands, weights and KV pools are bf16, or fp32 when the model is
@@ -93,7 +104,7 @@ from . import ops
 ARCHITECTURE = "Pumopel"
 # block style per architecture: how the norms sit around the sublayers (and which norm it is)
 BLOCK_STYLES = {"Pumopel": "dyt_sandwich", "Kenetar": "rms_post", "Zudarax": "rms_parallel", "Gerupel": "rms_dual",
-                "Goponex": "ln_post"}
+                "Goponex": "ln_post", "Natalorn": "rms_hyper"}
 ROT_ATTN_KINDS = ("attention", "attention_2", "attention_3")  # the parallel style's mixers
 _NO_WINDOW = 1 << 30
 
@@ -194,6 +205,9 @@ class LatentAttnSpec:
     q_rank: int
     scale: float
     rot: RotSpec = None
+    window: int = 0        # > 0: a query at position i sees keys i - window < j <= i
+    sink: bool = False     # a logit per head in the softmax denominator
+    gate_cols: bool = False  # the sigmoid output gate is per column of the concatenated heads, not per head
 
 
 @dataclass
@@ -302,8 +316,12 @@ class MoeSpec:
     # 'sigmoid_in': weights = sigmoid scores applied to the expert's input, clamped-swish experts;
     # 'softmax_out': weights = softmax over the chosen logits (+ router bias) applied to the experts' outputs, SiLU experts
     # 'softmax_renorm': weights = softmax over ALL experts, the chosen ones divided by their sum, times `scale`; on the outputs
+    # 'softmax_grouped': weights = softmax over ALL experts times `scale`, on the outputs; the choice is made on score + correction
+    # among the experts of the best `keep` of `groups` runs of neighbours
     route: str = "sigmoid_in"
     scale: float = 1.0
+    groups: int = 1
+    keep: int = 1
 
 
 @dataclass
@@ -331,8 +349,9 @@ class HybridConfig:
     logit_scale: float = 1.0
     norm_groups: int = 1         # parallel style: equal parts of a row that are normed on their own
     residual_mult: float = 1.0   # dual-norm style: factor on the sum of a layer's branches
-    loop: dict | None = None     # dual-norm style: start, stop, times -- layers [start, stop) run `times` times in a row
+    loop: dict | None = None     # dual-norm and hyper-connected styles: start, stop, times -- layers [start, stop) run `times` times
     postln_alpha: float = 1.0    # layer-norm-after-the-sum style: factor on x in the sum
+    streams: int = 1             # hyper-connected style: copies of the residual stream
 
     @property
     def style(self) -> str:
@@ -356,9 +375,12 @@ class HybridConfig:
         par = BLOCK_STYLES[name] == "rms_parallel"
         dual = BLOCK_STYLES[name] == "rms_dual"
         lnp = BLOCK_STYLES[name] == "ln_post"
+        hyp = BLOCK_STYLES[name] == "rms_hyper"
         for L in d["layers"]:
             m = L["mixer"]
-            if lnp:
+            if hyp:
+                mixer = _hyper_mixer(L["type"], m, name)
+            elif lnp:
                 mixer = _post_ln_mixer(L["type"], m, name)
             elif dual:
                 if L["type"] != "parallel":
@@ -394,13 +416,15 @@ class HybridConfig:
                     raise ValueError(f"latent attention: {mixer.rot.dims} rotating columns in a rotated part of {mixer.rot_dim}")
             else:
                 raise ValueError(f"unknown layer type {L['type']!r}")
-            if not par and not dual and not lnp and post != (L["type"] in ("delta", "latent_attention")):
+            if not par and not dual and not lnp and not hyp and post != (L["type"] in ("delta", "latent_attention")):
                 raise ValueError(f"layer type {L['type']!r} is not part of the {name} design")
             f = L.get("mlp")
             mlp = None
             if f:
                 kind = f.get("kind", "moe")
-                if lnp:
+                if hyp:
+                    mlp = _grouped_moe_spec(f)
+                elif lnp:
                     if kind != "dense":
                         raise ValueError(f"unknown feed-forward kind {kind!r}")
                     mlp = DenseSpec(int(f["ff"]), "relu2")
@@ -432,14 +456,17 @@ class HybridConfig:
         if int(d["width"]) % groups:
             raise ValueError(f"rows of {d['width']} do not split into {groups} equal norm groups")
         loop = None
-        if dual and d.get("loop"):
+        if (dual or hyp) and d.get("loop"):
             loop = {k: int(d["loop"][k]) for k in ("start", "stop", "times")}
             if not (0 <= loop["start"] < loop["stop"] <= len(layers) and loop["times"] >= 1):
                 raise ValueError(f"loop {loop} over {len(layers)} layers")
+        streams = int(d.get("streams") or 1) if hyp else 1
+        if not 1 <= streams <= 32:
+            raise ValueError(f"{streams} copies of the residual stream")
         return HybridConfig(int(d["vocab"]), int(d["width"]), float(d["norm"]["eps"]), float(emb.get("scale", 1.0)), layers, name,
                             {k: int(big[k]) for k in ("buckets", "mul_prev", "mul_cur")} if big else None,
                             float(d.get("logit_scale", 1.0)), groups, float(d.get("residual_mult", 1.0)) if dual else 1.0, loop,
-                            float(d["postln_alpha"]) if lnp else 1.0)
+                            float(d["postln_alpha"]) if lnp else 1.0, streams)
 
     @staticmethod
     def from_pretrained(path: str) -> "HybridConfig":
@@ -465,6 +492,11 @@ class HybridConfig:
         if self.style == "ln_post":
             del out["embedding"]
             out["postln_alpha"] = self.postln_alpha
+        if self.style == "rms_hyper":
+            del out["embedding"]
+            out["streams"] = self.streams
+            if self.loop:
+                out["loop"] = dict(self.loop)
         for L in self.layers:
             m = L.mixer
             if isinstance(m, DualMixerSpec):
@@ -484,10 +516,13 @@ class HybridConfig:
             elif isinstance(m, MatrixMemorySpec):
                 mixer = {"heads": m.heads, "dim": m.dim, "vdim": m.vdim, "gate_cap": m.gate_cap}
             elif isinstance(m, RotAttnSpec):
-                mixer = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale,
-                         "rot": {"dims": m.rot.dims, "base": m.rot.base}}
-                if m.rot.scaling:
-                    mixer["rot"]["scaling"] = dict(m.rot.scaling)
+                mixer = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "scale": m.scale}
+                if m.rot is not None:
+                    mixer["rot"] = {"dims": m.rot.dims, "base": m.rot.base}
+                    if m.rot.scaling:
+                        mixer["rot"]["scaling"] = dict(m.rot.scaling)
+                if m.window:
+                    mixer["mask"] = {"size": m.window}
                 if m.conv:
                     mixer["conv"] = m.conv
                 if m.chunk:
@@ -500,8 +535,11 @@ class HybridConfig:
                 mixer = {"heads": m.heads, "kv_heads": m.kv_heads, "dim": m.dim, "vdim": m.vdim, "conv": m.conv}
             elif L.kind == "latent_attention":
                 mixer = {"heads": m.heads, "dim": m.dim, "rot_dim": m.rot_dim, "vdim": m.vdim, "kv_rank": m.kv_rank,
-                         "q_rank": m.q_rank, "scale": m.scale,
-                         "rot": {"dims": m.rot.dims, "base": m.rot.base, "scaling": dict(m.rot.scaling) if m.rot.scaling else None}}
+                         "q_rank": m.q_rank, "scale": m.scale, "rot": {"dims": m.rot.dims, "base": m.rot.base}}
+                if self.style != "rms_hyper":
+                    mixer["rot"]["scaling"] = dict(m.rot.scaling) if m.rot.scaling else None
+                if m.window:
+                    mixer["mask"] = {"size": m.window}
             elif L.kind == "mamba2":
                 mixer = {"heads": m.heads, "vdim": m.vdim, "state": m.state, "groups": m.groups, "conv": m.conv,
                          "norm_groups": m.norm_groups}
@@ -513,6 +551,10 @@ class HybridConfig:
             f = None
             if isinstance(L.mlp, (DenseSpec, PolySpec)):
                 f = {"kind": "dense", "ff": L.mlp.ff}
+            elif L.mlp and L.mlp.route == "softmax_grouped":
+                f = {"kind": "moe", "router": {"experts": L.mlp.experts, "top": L.mlp.top, "scale": L.mlp.scale,
+                                               "groups": {"count": L.mlp.groups, "keep": L.mlp.keep}}, "expert": {"ff": L.mlp.ff},
+                     "shared": {"ff": L.mlp.shared_ff} if L.mlp.shared_ff else None}
             elif L.mlp and L.mlp.route == "softmax_renorm":
                 f = {"kind": "moe", "router": {"experts": L.mlp.experts, "top": L.mlp.top, "scale": L.mlp.scale}, "expert": {"ff": L.mlp.ff}}
             elif L.mlp and L.mlp.route == "softmax_out":
@@ -598,6 +640,42 @@ def _post_ln_mixer(kind: str, m: dict, name: str):
     return DualMixerSpec(left, right, 0.5, 0.5, branch_norm=True)
 
 
+def _hyper_mixer(kind: str, m: dict, name: str):
+    """One of the hyper-connected style's mixers from its configuration entry."""
+    size = int((m.get("mask") or {}).get("size") or 0)
+    if size < 0:
+        raise ValueError(f"{kind} layer: mask of {size}")
+    if kind in ("attention", "attention_2"):
+        spec = RotAttnSpec(int(m["heads"]), int(m["kv_heads"]), int(m["dim"]), int(m["vdim"]), float(m["scale"]))
+        if spec.heads % spec.kv_heads:
+            raise ValueError(f"{kind} layer: {spec.heads} query heads over {spec.kv_heads} kv heads")
+        if kind == "attention":
+            spec.window = size
+        else:
+            spec.bias, spec.chunk, spec.softcap = True, size, float(m.get("softcap") or 0.0)
+        return spec
+    if kind != "latent_attention":
+        raise ValueError(f"layer type {kind!r} is not part of the {name} design")
+    r = m["rot"]
+    spec = LatentAttnSpec(int(m["heads"]), int(m["dim"]), int(m["rot_dim"]), int(m["vdim"]), int(m["kv_rank"]), int(m["q_rank"]),
+                          float(m["scale"]), RotSpec(int(r["dims"]), float(r["base"])), window=size, sink=True, gate_cols=True)
+    if spec.rot.dims > spec.rot_dim or spec.rot.dims % 2:
+        raise ValueError(f"latent attention: {spec.rot.dims} rotating columns in a rotated part of {spec.rot_dim}")
+    return spec
+
+
+def _grouped_moe_spec(f: dict) -> MoeSpec:
+    """Experts behind a router that chooses inside the best groups of neighbours."""
+    if f.get("kind", "moe") != "moe":
+        raise ValueError(f"unknown feed-forward kind {f['kind']!r}")
+    r, g = f["router"], f["router"].get("groups") or {}
+    mlp = MoeSpec(int(r["experts"]), int(r["top"]), int(f["expert"]["ff"]), shared_ff=int((f.get("shared") or {}).get("ff") or 0),
+                  route="softmax_grouped", scale=float(r.get("scale", 1.0)), groups=int(g.get("count") or 1), keep=int(g.get("keep") or 1))
+    if mlp.experts % mlp.groups or not 1 <= mlp.keep <= mlp.groups or not 1 <= mlp.top <= mlp.keep * (mlp.experts // mlp.groups):
+        raise ValueError(f"router: top {mlp.top} of {mlp.experts} experts in {mlp.groups} groups of which {mlp.keep} are kept")
+    return mlp
+
+
 def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple]:
     """Checkpoint tensor name -> shape (a linear layer's matrix has one row per output)."""
     W = cfg.width
@@ -615,9 +693,10 @@ def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple]:
             s["loop.step"] = (cfg.loop["times"], W)
 
     lnp = cfg.style == "ln_post"
+    hyp = cfg.style == "rms_hyper"
 
     def norm(n):
-        if post or par or dual or lnp:
+        if post or par or dual or lnp or hyp:
             s[n] = (W,)
         else:
             s[n], s[n + ".b"], s[n + ".alpha"] = (W,), (W,), ()
@@ -625,9 +704,11 @@ def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple]:
     norm("final.norm")
     for i, L in enumerate(cfg.layers):
         p = f"l{i}."
-        for n in ("norm1",) if par else (("norm1",) + (("norm2",) if L.mlp else ())) if post or dual or lnp else \
+        for n in ("norm1",) if par else (("norm1",) + (("norm2",) if L.mlp else ())) if post or dual or lnp or hyp else \
                 (("norm1", "norm1b") + (("norm2", "norm2b") if L.mlp else ())):
             norm(p + n)
+        for q in (("hc1", "hc2") if L.mlp else ("hc1",)) if hyp else ():
+            s.update({f"{p}{q}.in": (cfg.streams,), f"{p}{q}.out": (cfg.streams,), f"{p}{q}.mix": (cfg.streams, cfg.streams)})
         m = L.mixer
         if isinstance(m, DualMixerSpec) and isinstance(m.right, MambaSpec):
             a, r = m.left, m.right
@@ -675,7 +756,10 @@ def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple]:
             s.update({p + "mix.dq": (m.q_rank, W), p + "mix.dq.norm": (m.q_rank,),
                       p + "mix.uq": (m.heads * (m.dim + m.rot_dim), m.q_rank), p + "mix.dkv": (m.kv_rank + m.rot_dim, W),
                       p + "mix.dkv.norm": (m.kv_rank,), p + "mix.uk": (m.heads * m.dim, m.kv_rank),
-                      p + "mix.uv": (m.heads * m.vdim, m.kv_rank), p + "mix.g": (m.heads, W), p + "mix.o": (W, m.heads * m.vdim)})
+                      p + "mix.uv": (m.heads * m.vdim, m.kv_rank), p + "mix.g": (m.heads * m.vdim if m.gate_cols else m.heads, W),
+                      p + "mix.o": (W, m.heads * m.vdim)})
+            if m.sink:
+                s[p + "mix.sink"] = (m.heads,)
         elif L.kind == "mamba2":
             s.update({p + "mix.in": (m.proj, W), p + "mix.conv": (m.channels, m.conv), p + "mix.conv.b": (m.channels,),
                       p + "mix.dt_bias": (m.heads,), p + "mix.A_log": (m.heads,), p + "mix.D": (m.heads,),
@@ -696,6 +780,8 @@ def tensor_shapes(cfg: HybridConfig) -> dict[str, tuple]:
             s[p + "mlp.router"] = (f.experts, W)
             if f.route == "softmax_out":
                 s[p + "mlp.router.b"] = (f.experts,)
+            if f.route == "softmax_grouped":
+                s[p + "mlp.correction"] = (f.experts,)
             for e in range(f.experts):
                 s.update({f"{p}mlp.e{e}.gate": (f.ff, W), f"{p}mlp.e{e}.up": (f.ff, W), f"{p}mlp.e{e}.down": (W, f.ff)})
             if f.shared_ff:
@@ -721,6 +807,10 @@ def random_weights(cfg: HybridConfig, seed: int = 0, std: float | None = None) -
             t = 0.6 + 0.8 * torch.rand(shape, generator=g)
         elif leaf == "lower":
             t = 0.9 * torch.rand(shape, generator=g)
+        elif cfg.style == "rms_hyper" and leaf == "in":
+            t = (1.0 + 0.4 * torch.randn(shape, generator=g)) / shape[0]
+        elif cfg.style == "rms_hyper" and leaf == "mix":
+            t = 0.9 * torch.eye(shape[0]) + 0.25 * torch.randn(shape, generator=g) / shape[0] ** 0.5
         elif leaf == "step":
             t = 0.2 * torch.randn(shape, generator=g)
         elif cfg.style == "ln_post" and name.endswith(".dt.b"):
@@ -867,9 +957,10 @@ class HybridCausalLM:
         par = cfg.style == "rms_parallel"
         dual = cfg.style == "rms_dual"
         lnp = cfg.style == "ln_post"
+        hyp = cfg.style == "rms_hyper"
 
         def norm(name):
-            if post or par or dual or lnp:  # weight stored around zero (post-norm) or plain (RMS in groups: parallel; layer norm)
+            if post or par or dual or lnp or hyp:  # weight stored around zero (post-norm) or plain (RMS in groups: parallel; layer norm)
                 return vec(name)
             return (vec(name), vec(name + ".b"), float(get(name + ".alpha").float()))
 
@@ -892,7 +983,7 @@ class HybridCausalLM:
         for i, L in enumerate(cfg.layers):
             p, m = f"l{i}.", L.mixer
             lw = {"spec": L, "norm1": norm(p + "norm1")}
-            if not post and not par and not dual and not lnp:
+            if not post and not par and not dual and not lnp and not hyp:
                 lw["norm1b"] = norm(p + "norm1b")
             if isinstance(m, DualMixerSpec) and isinstance(m.right, MambaSpec):
                 a, r = m.left, m.right
@@ -937,6 +1028,10 @@ class HybridCausalLM:
                           w_o=lin(p + "mix.left.o"), w_o2=lin(p + "mix.right.o"), temp=vec(p + "mix.left.temp"),
                           sink=torch.zeros((a.heads,), dtype=torch.float32, device=dev),  # exp(0) = the 1 in the denominator
                           f_bias=vec(p + "mix.right.f.b"), lower=vec(p + "mix.right.lower"), onorm=vec(p + "mix.right.norm"))
+            elif isinstance(m, RotAttnSpec) and m.rot is None:
+                lw.update(w_in=lin(p + "mix.q", p + "mix.k", p + "mix.v"), w_o=lin(p + "mix.o"))
+                if m.bias:
+                    lw["in_bias"] = torch.cat([get(p + f"mix.{n}.b") for n in "qkv"]).to(dev, torch.float32).contiguous()
             elif isinstance(m, RotAttnSpec):
                 key = (m.rot.dims, m.rot.base, json.dumps(m.rot.scaling, sort_keys=True))
                 if key not in rot_tables:
@@ -981,8 +1076,11 @@ class HybridCausalLM:
                           dkv_norm=vec(p + "mix.dkv.norm"), w_uq=lin(p + "mix.uq"), w_o=lin(p + "mix.o"), rot=rot_tables[key],
                           # per head: the key up-projection transposed (it is folded into the query), the value up-projection
                           w_absorb=get(p + "mix.uk").view(m.heads, m.dim, m.kv_rank).transpose(1, 2).to(dev, et).contiguous(),
-                          w_uv=get(p + "mix.uv").view(m.heads, m.vdim, m.kv_rank).to(dev, et).contiguous(),
-                          k_pool=torch.zeros((num_blocks, 1, block_size, m.kv_rank + m.rot_dim), dtype=et, device=dev))
+                          w_uv=get(p + "mix.uv").view(m.heads, m.vdim, m.kv_rank).to(dev, et).contiguous())
+                if m.sink:
+                    lw["sink"] = vec(p + "mix.sink")
+                if not hyp:
+                    lw["k_pool"] = torch.zeros((num_blocks, 1, block_size, m.kv_rank + m.rot_dim), dtype=et, device=dev)
             elif L.kind == "mamba2":
                 lw.update(w_in=lin(p + "mix.in"), conv_w=vec(p + "mix.conv"), conv_b=vec(p + "mix.conv.b"),
                           dt_bias=vec(p + "mix.dt_bias"), a_log=vec(p + "mix.A_log"), d=vec(p + "mix.D"),
@@ -1004,9 +1102,12 @@ class HybridCausalLM:
                         raise ValueError("value mixing needs the same kv_heads * vdim in every v_mix layer")
                     first_vmix = False
             f = L.mlp
+            if hyp:
+                for q in ("hc1", "hc2") if f else ("hc1",):
+                    lw[q] = {n: vec(f"{p}{q}.{n}") for n in ("in", "mix", "out")}
             if f and not par:
                 lw["norm2"] = norm(p + "norm2")
-                if not post and not dual and not lnp:
+                if not post and not dual and not lnp and not hyp:
                     lw["norm2b"] = norm(p + "norm2b")
             if isinstance(f, PolySpec):  # W_up rides in w_in
                 lw.update(w_down=lin(p + "mlp.down"), act=vec(p + "mlp.act"))
@@ -1018,6 +1119,8 @@ class HybridCausalLM:
                 lw["w_router"] = lin(p + "mlp.router")
                 if f.route == "softmax_out":
                     lw["router_b"] = vec(p + "mlp.router.b")
+                if f.route == "softmax_grouped":
+                    lw["correction"] = vec(p + "mlp.correction")
                 lw["w_gu"] = torch.stack([torch.cat([get(f"{p}mlp.e{e}.gate"), get(f"{p}mlp.e{e}.up")]) for e in range(f.experts)]
                                          ).to(dev, et).contiguous()
                 lw["w_down"] = torch.stack([get(f"{p}mlp.e{e}.down") for e in range(f.experts)]).to(dev, et).contiguous()
@@ -1025,7 +1128,7 @@ class HybridCausalLM:
                     lw["sh_gu"] = lin(p + "mlp.shared.gate", p + "mlp.shared.up")
                     lw["sh_down"] = lin(p + "mlp.shared.down")
             self.layers.append(lw)
-        # dual-norm style: one entry per layer RUN (a repeated layer runs loop.times times with the same weights); every run has
+        # dual-norm and hyper-connected styles: one entry per layer RUN (a repeated layer runs loop.times times with the same weights); every run has
         # K / V pools, pooled-block pools and recurrent state of its own
         self.runs = []
         if dual:
@@ -1040,6 +1143,17 @@ class HybridCausalLM:
                     run.update(pk_pool=torch.zeros((num_blocks, a.kv_heads, ppb, a.dim), dtype=et, device=dev),
                                pv_pool=torch.zeros((num_blocks, a.kv_heads, ppb, a.vdim), dtype=et, device=dev))
                 self.runs.append(run)
+        if hyp:
+            self.read_all = torch.ones((cfg.streams,), dtype=torch.float32, device=dev)  # the logits read the sum of the copies
+            for i, rep in cfg.layer_runs():
+                m = cfg.layers[i].mixer
+                pool = lambda heads, cols: torch.zeros((num_blocks, heads, block_size, cols), dtype=et, device=dev)  # noqa: E731
+                run = {"lw": self.layers[i], "layer": i, "rep": rep}
+                if isinstance(m, LatentAttnSpec):
+                    run["k_pool"] = pool(1, m.kv_rank + m.rot_dim)
+                else:
+                    run.update(k_pool=pool(m.kv_heads, m.dim), v_pool=pool(m.kv_heads, m.vdim))
+                self.runs.append(run)
         self.block_table = torch.zeros((slots, self.max_blocks), dtype=torch.int32, device=dev)
         self.num_tokens = torch.zeros((slots,), dtype=torch.int32, device=dev)
         self.gemm_ws = None
@@ -1049,7 +1163,7 @@ class HybridCausalLM:
     # ------------------------------------------------------------------ sizes
     def kv_bytes_per_block(self) -> int:
         es = 2 if self.et == torch.bfloat16 else 4
-        if self.cfg.style == "rms_dual":  # per run: K / V rows of a page and its pooled-block rows
+        if self.cfg.style in ("rms_dual", "rms_hyper"):  # per run: K / V rows of a page and its pooled-block rows
             return sum(sum(t.shape[1] * t.shape[2] * t.shape[3] * es for n, t in run.items() if n.endswith("_pool")) for run in self.runs)
         if self.cfg.style == "ln_post":
             return sum(L.mixer.left.kv_heads * self.block_size * (L.mixer.left.dim + L.mixer.left.vdim) * es
@@ -1059,6 +1173,8 @@ class HybridCausalLM:
             sum(self.block_size * (L.mixer.kv_rank + L.mixer.rot_dim) * es for L in self.cfg.layers if L.kind == "latent_attention")
 
     def state_bytes_per_slot(self) -> int:
+        if self.cfg.style == "rms_hyper":
+            return 0
         if self.cfg.style == "rms_dual":
             return sum(4 * run["scan_state"][0].numel() for run in self.runs)
         if self.cfg.style == "ln_post":
@@ -1116,22 +1232,23 @@ class HybridCausalLM:
                            m.dim, m.vdim, m.dim ** -0.5)
         return self._linear(ops.head_rmsnorm_gate(o, proj, c + 2 * m.heads, lw["onorm"], self.cfg.eps, m.heads, self.et), lw["w_o"])
 
-    def _latent_attention(self, lw, h, meta):
+    def _latent_attention(self, lw, h, meta, pool=None):
         m = lw["spec"].mixer
+        pool = lw["k_pool"] if pool is None else pool
         cos, sin = lw["rot"]
         kr = m.kv_rank + m.rot_dim
         proj = self._linear(h, lw["w_in"])  # fp32 [T, query latent | kv latent | shared rotated key part | head gates]
         ops.latent_kv_write(proj, m.q_rank, m.kv_rank, m.rot_dim, m.rot.dims, lw["dkv_norm"], self.cfg.eps, cos, sin, meta,
-                            lw["k_pool"])
+                            pool)
         cq = ops.rmsnorm_cols(proj, 0, m.q_rank, lw["dq_norm"], self.cfg.eps, self.et)
         q = self._linear(cq, lw["w_uq"])  # fp32 [T, H * (dim + rot_dim)]
         nope, q_att = ops.latent_q_prep(q, m.heads, m.dim, m.rot_dim, m.rot.dims, m.kv_rank, cos, sin, meta, self.et)
         ops.batched_linear(nope, lw["w_absorb"], q_att, a_batch_stride=m.dim, out_batch_stride=kr)
-        lat = ops.swa_sink_attn(q_att, m.heads, lw["k_pool"], None, self.block_table, meta, None, m.scale, _NO_WINDOW,
+        lat = ops.swa_sink_attn(q_att, m.heads, pool, None, self.block_table, meta, lw.get("sink"), m.scale, m.window or _NO_WINDOW,
                                 latent_values=m.kv_rank)  # [T, H * kv_rank]
         vals = torch.empty((h.shape[0], m.heads * m.vdim), dtype=self.et, device=self.device)
         ops.batched_linear(lat, lw["w_uv"], vals, a_batch_stride=m.kv_rank, out_batch_stride=m.vdim,
-                           gate=proj[:, m.q_rank + kr:])
+                           gate=proj[:, m.q_rank + kr:], gate_cols=m.gate_cols)
         return self._linear(vals, lw["w_o"])
 
     def _rot_attention(self, lw, proj, meta):
@@ -1300,6 +1417,64 @@ class HybridCausalLM:
         self.last_logits = self._linear(hf, self.head)
         return self.last_logits
 
+    def _plain_attention(self, run, h, meta):
+        """Attention without rotation: a sliding window, or biased projections, capped scores and chunks."""
+        lw = run["lw"]
+        m = lw["spec"].mixer
+        proj = self._linear(h, lw["w_in"])  # fp32 [T, q | k | v]
+        k0, v0 = m.q_cols, m.q_cols + m.k_cols
+        if m.bias:
+            q = ops.qk_norm_rope_kv_write(proj, 0, k0, v0, m.heads, run["k_pool"], run["v_pool"], meta, bias=lw["in_bias"])
+        else:  # the projection rows are the queries as they are
+            ops.kv_write_vmix(proj, k0, v0, run["k_pool"], run["v_pool"], meta.slot_mapping)
+            q = proj
+        a = ops.swa_sink_attn(q, m.heads, run["k_pool"], run["v_pool"], self.block_table, meta, None, m.scale, m.window or _NO_WINDOW,
+                              chunk=m.chunk, softcap=m.softcap, split_p=True)
+        return self._linear(a, lw["w_o"])
+
+    def _grouped_moe(self, lw, h):
+        """-> (shared expert's rows or None, the chosen experts' rows, their weights)."""
+        f = lw["spec"].mlp
+        idx, wt = ops.moe_topk_grouped(self._linear(h, lw["w_router"]), lw["correction"], f.top, groups=f.groups, keep=f.keep, scale=f.scale)
+        align = ops.moe_align(idx, f.experts, ops.moe_wide_tiles(h, lw["w_gu"], idx.numel()))
+        pairs = ops.moe_experts(h, wt, align, lw["w_gu"], lw["w_down"], f.top, act=ops.ACT_SILU, scale_input=False)
+        shared = None
+        if f.shared_ff:
+            shared = self._linear(ops.glu(self._linear(h, lw["sh_gu"]), ops.ACT_SILU, self.et), lw["sh_down"])
+        return shared, pairs, wt
+
+    def _forward_hyper(self, tokens, meta, logit_rows, capture):
+        """u = sum_s r_s x_s; y = sublayer(N(u)); x_t <- sum_s M[s, t] x_s + o_t y: one pass over the copies per sublayer adds its
+        output (the experts' rows weighed on the way), mixes, and writes the next sublayer's normed input."""
+        et, cfg, runs = self.et, self.cfg, self.runs
+
+        def entering(k):  # read vector and norm weight of the sublayer that comes first in run k (or of the logits)
+            return (runs[k]["lw"]["hc1"]["in"], runs[k]["lw"]["norm1"]) if k < len(runs) else (self.read_all, self.final_norm)
+
+        x, h = ops.hyper_embed(tokens, self.embed, cfg.streams, *entering(0), cfg.eps)
+        for k, run in enumerate(runs):
+            lw = run["lw"]
+            f, c1 = lw["spec"].mlp, lw["hc1"]
+            keep = dict(out_dtype=et, store=k + 1 < len(runs) or capture is not None)  # nothing reads the copies after the last sublayer
+            if isinstance(lw["spec"].mixer, LatentAttnSpec):
+                y = self._latent_attention(lw, h, meta, run["k_pool"])
+            else:
+                y = self._plain_attention(run, h, meta)
+            if f:
+                c2 = lw["hc2"]
+                h = ops.hyper_residual(x, c1["mix"], c1["out"], c2["in"], lw["norm2"], cfg.eps, y1=y, out_dtype=et)
+                shared, pairs, wt = self._grouped_moe(lw, h)
+                h = ops.hyper_residual(x, c2["mix"], c2["out"], *entering(k + 1), cfg.eps, y1=shared, y2=pairs, nsum=f.top, y2_weight=wt, **keep)
+            else:
+                h = ops.hyper_residual(x, c1["mix"], c1["out"], *entering(k + 1), cfg.eps, y1=y, **keep)
+            if capture is not None:
+                capture.append(x.sum(1))
+        if logit_rows is None or logit_rows.numel() == 0:
+            self.last_logits = None
+            return None
+        self.last_logits = self._linear(h.index_select(0, logit_rows).contiguous(), self.head)
+        return self.last_logits
+
     def _post_ff(self, lw, h):
         """Feed-forward of the post-norm style -> (fp32 branch rows, rows per token, their weights or None)."""
         f = lw["spec"].mlp
@@ -1353,6 +1528,8 @@ class HybridCausalLM:
             return self._forward_parallel(tokens, meta, logit_rows, capture)
         if self.cfg.style == "ln_post":
             return self._forward_post_ln(tokens, meta, logit_rows, capture)
+        if self.cfg.style == "rms_hyper":
+            return self._forward_hyper(tokens, meta, logit_rows, capture)
         if self.cfg.style == "rms_dual":
             return self._forward_dual(tokens, meta, logit_rows, capture)
         et, n = self.et, len(self.layers)

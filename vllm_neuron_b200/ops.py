@@ -777,7 +777,7 @@ def swa_sink_attn(q_src, num_heads: int, k_pool, v_pool, block_table, meta, sink
     variant = (int(chunk), float(softcap), _ptr(sigmoid_bias), v_div, 1 if out_f32 else 0)
     plain = not chunk and not softcap and sigmoid_bias is None and v_div == 1 and not out_f32
     # the per-launch timer tells the variants apart (their floors differ)
-    tag = "" if plain and not pool and not keep else "[" + "+".join(n for n, on in (("chunk", chunk), ("cap", softcap), ("sigmoid", sigmoid_bias is not None),
+    tag = "[latent]" if plain and latent_values else "" if plain and not pool and not keep else "[" + "+".join(n for n, on in (("chunk", chunk), ("cap", softcap), ("sigmoid", sigmoid_bias is not None),
                                                                        ("maps", v_div > 1), ("pool", pool), ("keep", keep)) if on) + "]"
     # long prompt portions in bf16 serving (a sliding window only without pooled blocks), head sizes of 64 / 128 with pages of 32 tokens: the tcgen05 kernel (128-row query
     # tiles, accumulators in tensor memory); B200_SWA_PREFILL_LEGACY=1 keeps the mma.sync kernel (A/B aid)
@@ -806,13 +806,14 @@ def swa_sink_attn(q_src, num_heads: int, k_pool, v_pool, block_table, meta, sink
                                                           1 if split_p else 0, *pool_args, _stream()),
                   "b200_swa_sink_attn_prefill")
         return out
-    if (plain and latent_values and sink is None and window >= (1 << 30) and k_pool.dtype == torch.bfloat16 and d % 16 == 0 and dv % 16 == 0
+    if (plain and latent_values and k_pool.dtype == torch.bfloat16 and d % 16 == 0 and dv % 16 == 0
             and dv <= 256 and q_src.stride(0) % 2 == 0):
         # attention over cached latents, decode-sized steps: the heads of a token are the rows of a tensor-core tile
         with _k("latent_attn_decode"):
             check(_cabi.load().b200_latent_attn_decode(_ptr(q_src), q_src.stride(0), _ptr(k_pool), _ptr(block_table),
-                                                       block_table.stride(0), _ptr(meta.tok_row), _ptr(meta.tok_pos), float(scale),
-                                                       _ptr(out), t, num_heads, d, dv, bs, _stream()), "b200_latent_attn_decode")
+                                                       block_table.stride(0), _ptr(meta.tok_row), _ptr(meta.tok_pos), _ptr(sink),
+                                                       float(scale), int(window), _ptr(out), t, num_heads, d, dv, bs, _stream()),
+                  "b200_latent_attn_decode")
         return out
     # long contexts at small batch: several CTAs share a (token, kv head)'s keys, so that every SM has its CTAs
     span = min(getattr(meta, "max_end", 0) or 0, int(window), int(chunk) if chunk else 1 << 30)
@@ -854,6 +855,23 @@ def moe_topk(logits, top: int, bias=None, mode: int = ROUTE_SIGMOID):
     with _k("moe_topk"):
         check(_cabi.load().b200_moe_topk(_ptr(logits), logits.stride(0), _ptr(bias), int(mode), _ptr(idx), _ptr(wt), t, e, top,
                                          _stream()), "b200_moe_topk")
+    return idx, wt
+
+
+def moe_topk_grouped(logits, correction, top: int, *, groups: int = 1, keep: int = 1, scale: float = 1.0):
+    """fp32 router logits [T, E] -> (expert ids int32 [T, top], routing weights fp32 [T, top]).  Scores = softmax over all experts;
+    the `top` largest of score + correction (fp32 [E] or None) are chosen among the experts of the best `keep` of `groups` equal
+    runs of neighbours (a run's rank: its largest choice score); weight = score * scale."""
+    _cuda(logits, correction)
+    _f32(correction)
+    assert logits.dtype == torch.float32 and logits.stride(1) == 1
+    t, e = logits.shape
+    assert correction is None or correction.numel() == e
+    idx = torch.empty((t, top), dtype=torch.int32, device=logits.device)
+    wt = torch.empty((t, top), dtype=torch.float32, device=logits.device)
+    with _k("moe_topk_grouped"):
+        check(_cabi.load().b200_moe_topk_grouped(_ptr(logits), logits.stride(0), _ptr(correction), int(groups), int(keep), float(scale),
+                                                 _ptr(idx), _ptr(wt), t, e, top, _stream()), "b200_moe_topk_grouped")
     return idx, wt
 
 
@@ -901,10 +919,10 @@ def linear_simt(a, w):
     return out
 
 
-def batched_linear(a, w, out, *, a_batch_stride: int, out_batch_stride: int, gate=None):
+def batched_linear(a, w, out, *, a_batch_stride: int, out_batch_stride: int, gate=None, gate_cols: bool = False):
     """out_b = a_b @ w[b]^T for every b of w [batch, N, K] in one launch: a_b = rows of `a` (pitch a.stride(0)) starting at
     column b * a_batch_stride, out_b likewise in `out` (fp32, or the operand type).  gate: fp32 view [M, >= batch] whose
-    sigmoid multiplies out_b's rows."""
+    sigmoid multiplies out_b's rows -- or, with gate_cols, [M, >= batch * N], a gate per output column (column b * N + n)."""
     _cuda(a, w, out, gate)
     assert a.dtype == w.dtype and a.stride(1) == 1 and out.stride(1) == 1 and w.is_contiguous() and w.dim() == 3
     b, n, k = w.shape
@@ -913,10 +931,12 @@ def batched_linear(a, w, out, *, a_batch_stride: int, out_batch_stride: int, gat
     assert typed or out.dtype == torch.float32
     if gate is not None:
         assert gate.dtype == torch.float32 and gate.stride(1) == 1 and gate.shape[0] == m
+        assert gate.shape[1] >= (b * n if gate_cols else b)
     with _k(f"batched_linear[{b}x{m}x{n}x{k}]"):
         check(_cabi.load().b200_batched_linear(_ptr(a), a.stride(0), a_batch_stride, _ptr(w), n * k, _ptr(out), out.stride(0),
                                                out_batch_stride, b, m, n, k, _edt(a), 1 if typed else 0, _ptr(gate),
-                                               gate.stride(0) if gate is not None else 0, _stream()), "b200_batched_linear")
+                                               gate.stride(0) if gate is not None else 0, 1 if gate_cols and gate is not None else 0, _stream()),
+              "b200_batched_linear")
     return out
 
 
@@ -1127,15 +1147,16 @@ def diff_head_norm_gate(a, lam: float, post: float, gate_src, gate_col0: int, ep
 
 def qk_norm_rope_kv_write(src, q_col0: int, k_col0: int, v_col0: int, heads: int, k_pool, v_pool, meta, *, q_norm=None,
                           k_norm=None, eps: float = 0.0, rot_n: int = 0, rot_half: bool = True, cos=None, sin=None, q_head_scale=None,
-                          head_norm: bool = False):
+                          head_norm: bool = False, bias=None):
     """fp32 rows src = [.. q: heads * D .. k: G * D .. v: Gv * Dv ..] -> q fp32 [T, heads * D] (normed over the whole projection
     when q_norm is given, leading rot_n columns of every head rotated by the token's position), and the step's keys (same
     treatment) and values written into the pools [num_blocks, G, block_size, D] / [num_blocks, Gv, block_size, Dv].
     q_head_scale fp32 [heads]: q of head h is multiplied by it (a per-head temperature of the scores).
     head_norm: the norms are per head, q_norm / k_norm fp32 [D] shared by the heads.  v_col0 may equal k_col0: the cached values
-    are then the keys as projected, before norm and rotation."""
-    _cuda(src, k_pool, v_pool, q_norm, k_norm, cos, sin, q_head_scale)
-    _f32(q_norm, k_norm, cos, sin, q_head_scale)
+    are then the keys as projected, before norm and rotation.  bias fp32 [heads * D + G * D + Gv * Dv]: the projections' biases,
+    q | k | v, added ahead of everything else."""
+    _cuda(src, k_pool, v_pool, q_norm, k_norm, cos, sin, q_head_scale, bias)
+    _f32(q_norm, k_norm, cos, sin, q_head_scale, bias)
     assert q_head_scale is None or q_head_scale.numel() == heads
     assert src.dtype == torch.float32 and src.stride(1) == 1 and k_pool.dtype == v_pool.dtype
     assert k_pool.is_contiguous() and v_pool.is_contiguous()
@@ -1144,6 +1165,7 @@ def qk_norm_rope_kv_write(src, q_col0: int, k_col0: int, v_col0: int, heads: int
     assert rot_n == 0 or (cos.shape[1] == rot_n // 2 and sin.shape == cos.shape)
     assert q_norm is None or q_norm.numel() == (d if head_norm else heads * d)
     assert k_norm is None or k_norm.numel() == (d if head_norm else g * d)
+    assert bias is None or bias.numel() == (heads + g) * d + gv * dv
     t = src.shape[0]
     q = torch.empty((t, heads * d), dtype=torch.float32, device=src.device)
     with _k("qk_norm_rope_kv_write"):
@@ -1151,7 +1173,7 @@ def qk_norm_rope_kv_write(src, q_col0: int, k_col0: int, v_col0: int, heads: int
                                                       float(eps), int(rot_n), 1 if rot_half else 0, _ptr(cos), _ptr(sin),
                                                       _ptr(meta.tok_pos), _ptr(meta.slot_mapping), _ptr(q), _ptr(k_pool),
                                                       _ptr(v_pool), _edt(k_pool), t, heads, g, gv, d, dv, bs, _ptr(q_head_scale),
-                                                      1 if head_norm else 0, _stream()),
+                                                      1 if head_norm else 0, _ptr(bias), _stream()),
               "b200_qk_norm_rope_kv_write")
     return q
 
@@ -1368,4 +1390,38 @@ def bias_act(src, col0: int, n: int, bias, act: int, out_dtype):
     with _k("bias_act[relu2]" if act == ACT_RELU2 else "bias_act"):
         check(_cabi.load().b200_bias_act(_ptr(src), src.stride(0), col0, n, _ptr(bias), int(act), _ptr(out), _edt(out), t, _stream()),
               "b200_bias_act")
+    return out
+
+
+# ------------------------------------------------------------------ hyper-connected decoders (several copies of the residual stream)
+def hyper_embed(tokens, table, streams: int, read, w, eps: float):
+    """tokens int32 [T] -> (x fp32 [T, streams, W], every copy = table[token]; the RMS norm of sum_s read[s] x_s times w in the
+    table's type: the first sublayer's input)."""
+    _cuda(tokens, table, read, w)
+    _f32(read, w)
+    assert tokens.dtype == torch.int32 and table.is_contiguous() and read.numel() == streams
+    t, (v, width) = tokens.numel(), table.shape
+    x = torch.empty((t, streams, width), dtype=torch.float32, device=table.device)
+    out = torch.empty((t, width), dtype=table.dtype, device=table.device)
+    with _k("hyper_embed"):
+        check(_cabi.load().b200_hyper_embed(_ptr(tokens), _ptr(table), _edt(table), _ptr(x), streams, _ptr(read), _ptr(w), float(eps),
+                                            _ptr(out), t, width, v, _stream()), "b200_hyper_embed")
+    return x, out
+
+
+def hyper_residual(x, mix, write, read, w, eps: float, *, y1=None, y2=None, nsum: int = 1, y2_weight=None, out_dtype, store: bool = True):
+    """One sublayer's output joins the copies x fp32 [T, S, W]: with y = y1 + sum_c y2_weight[t, c] y2[t nsum + c],
+    x_d <- sum_s mix[s, d] x_s + write[d] y (in place unless store is False); returns the RMS norm of sum_d read[d] x_d of the new
+    copies, times w, in out_dtype (the next sublayer's input)."""
+    _cuda(x, mix, write, read, w, y1, y2, y2_weight)
+    _f32(x, mix, write, read, w, y2, y2_weight)
+    t, s, width = x.shape
+    assert mix.shape == (s, s) and write.numel() == s and read.numel() == s and w.numel() == width
+    assert y1 is None or (y1.dtype == torch.float32 and y1.stride(1) == 1 and y1.shape == (t, width))
+    assert y2 is None or (y2.shape == (t * nsum, width) and (y2_weight is None or y2_weight.numel() == t * nsum))
+    out = torch.empty((t, width), dtype=out_dtype, device=x.device)
+    with _k("hyper_residual" + ("" if y2 is None else "[experts]")):
+        check(_cabi.load().b200_hyper_residual(_ptr(x), s, _ptr(y1), y1.stride(0) if y1 is not None else 0, _ptr(y2), int(nsum),
+                                               _ptr(y2_weight), _ptr(mix), _ptr(write), _ptr(read), _ptr(w), float(eps),
+                                               1 if store else 0, _ptr(out), _edt(out), t, width, _stream()), "b200_hyper_residual")
     return out

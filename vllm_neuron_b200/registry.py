@@ -11,7 +11,8 @@ Two families are served:
     "Gerupel": parallel branches behind two RMS norms, a mixer that is windowed attention with pooled far blocks beside a gated
     linear recurrence, repeated layer runs with shared weights, MoE, logits from the embedding table; "Goponex": layer norm after
     the sum, a mixer that is windowed attention with kept first tokens (values = keys) beside a selective scan with a step size per
-    channel, matrix-memory layers, squared-relu feed-forward.
+    channel, matrix-memory layers, squared-relu feed-forward; "Natalorn": hyper-connections (several copies of the residual stream)
+    around windowed, chunked and latent attention, grouped-router MoE with a shared expert, repeated layer runs.
 The reference resolves the architecture the same way -- `hf_config.architectures[0]` picks the NxDI model class
 (vllm_neuron/worker/neuronx_distributed_model_loader.py:612-660).
 """
@@ -82,6 +83,7 @@ MODEL_REGISTRY: dict[str, ModelEntry] = {
     "Zudarax": ModelEntry("hybrid", _hybrid_config, _hybrid_weights, _hybrid_build, (torch.bfloat16, torch.float32)),
     "Gerupel": ModelEntry("hybrid", _hybrid_config, _hybrid_weights, _hybrid_build, (torch.bfloat16, torch.float32)),
     "Goponex": ModelEntry("hybrid", _hybrid_config, _hybrid_weights, _hybrid_build, (torch.bfloat16, torch.float32)),
+    "Natalorn": ModelEntry("hybrid", _hybrid_config, _hybrid_weights, _hybrid_build, (torch.bfloat16, torch.float32)),
 }
 
 

@@ -717,13 +717,14 @@ def main():
     ap.add_argument("--attn-traffic", type=float, default=None,
                     help="dram bytes read+written per attention launch from the committed ncu --set full capture")
     ap.add_argument("--hybrid", default="", choices=["", "small", "1b", "all", "kenetar-small", "kenetar-1b", "zudarax-small", "zudarax-1b",
-                                                       "gerupel-small", "gerupel-1b", "goponex-small", "goponex-1b"],
+                                                       "gerupel-small", "gerupel-1b", "goponex-small", "goponex-1b", "natalorn-small", "natalorn-1b"],
                     help="instead of the headline workload: prefill / decode throughput and per-kernel floors of the hybrid "
                          "(state-space + windowed attention + MoE) decoder beside the dense decoder at equal size, or (kenetar-*) of "
                          "the delta-rule + latent-attention decoder beside that hybrid at equal size, or (zudarax-*) of the parallel-branch "
                          "decoder with chunked / differential / sigmoid attention beside the dense decoder, or (gerupel-*) of the "
                          "dual-norm parallel decoder (window + pooled-block attention beside a gated recurrence) beside that hybrid, or (goponex-*) of the "
-                         "layer-norm-after-the-sum decoder (kept-token attention beside a selective scan, matrix memory) beside both; "
+                         "layer-norm-after-the-sum decoder (kept-token attention beside a selective scan, matrix memory) beside both, or (natalorn-*) of the hyper-connected decoder "
+                         "(windowed / chunked / latent attention, grouped-router experts) beside the delta-rule, the parallel-branch and the state-space decoders; "
                          "one JSON line per size "
                          "(vllm_neuron_b200/hybrid_bench.py)")
     args = ap.parse_args()

@@ -155,9 +155,10 @@ __global__ void hyper_residual_kernel(float* __restrict__ x, int S, const float*
   hc_norm_row<OT, V>(row, ss, w, eps, out + t * W, W);
 }
 
-static int hc_threads(int W, bool v4) {
+// many tokens: small CTAs, so that several rows per SM are in different phases; few tokens: more threads on each row
+static int hc_threads(int T, int W, bool v4) {
   const int per = v4 ? W / 4 : W;
-  return per > 256 ? 512 : per > 128 ? 256 : per > 64 ? 128 : 64;
+  return T >= 512 || per <= 128 ? 128 : 256;
 }
 
 }  // namespace b200
@@ -179,7 +180,7 @@ int b200_hyper_embed(const int32_t* tokens, const void* table, int dtype, float*
   B200_DISPATCH_ELEM(dtype, ET, {                                                                                                \
     if (smem > 48 * 1024)                                                                                                        \
       B200_CUDA_OK(cudaFuncSetAttribute(hyper_embed_kernel<ET, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));     \
-    B200_CUDA_OK(launch_kernel(hyper_embed_kernel<ET, V>, dim3(T), dim3(hc_threads(W, V == 4)), smem, (cudaStream_t)stream, tokens, \
+    B200_CUDA_OK(launch_kernel(hyper_embed_kernel<ET, V>, dim3(T), dim3(hc_threads(T, W, V == 4)), smem, (cudaStream_t)stream, tokens, \
                                (const ET*)table, x, S, read, w, eps, (ET*)out, W, vocab));                                       \
   })
   if (v4) HC_EMBED(4);
@@ -202,7 +203,7 @@ int b200_hyper_residual(float* x, int S, const float* y1, int ld1, const float* 
   B200_DISPATCH_ELEM(out_dtype, OT, {                                                                                               \
     if (smem > 48 * 1024)                                                                                                           \
       B200_CUDA_OK(cudaFuncSetAttribute(hyper_residual_kernel<OT, NS, V>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
-    B200_CUDA_OK(launch_kernel(hyper_residual_kernel<OT, NS, V>, dim3(T), dim3(hc_threads(W, V == 4)), smem, (cudaStream_t)stream, x, \
+    B200_CUDA_OK(launch_kernel(hyper_residual_kernel<OT, NS, V>, dim3(T), dim3(hc_threads(T, W, V == 4)), smem, (cudaStream_t)stream, x, \
                                S, y1, ld1, y2, nsum, y2_weight, mix, write, read, w, eps, store, (OT*)out, W));                     \
   })
 #define HC_PICK(NS)                \

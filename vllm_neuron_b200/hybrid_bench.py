@@ -3,7 +3,8 @@ at equal size (`small`, `1b`), the Kenetar design next to Pumopel at equal size 
 Zudarax design next to the dense Llama decoder at equal size (`zudarax-small`, `zudarax-1b`), and the Gerupel design next to
 Pumopel (its closest relative: windowed sink attention, a recurrence, experts) at equal size (`gerupel-small`, `gerupel-1b`),
 and the Goponex design next to Gerupel (windowed attention beside a recurrence) and Pumopel (a state-space scan) at equal size
-(`goponex-small`, `goponex-1b`).
+(`goponex-small`, `goponex-1b`), and the Natalorn design next to Kenetar (latent attention, experts), Zudarax (chunked capped
+attention) and Pumopel (windowed attention, a shared expert) at equal size (`natalorn-small`, `natalorn-1b`).
 
 For each size: random weights, both models in bf16 on one GPU, same width / layer count / vocabulary; the dense model's
 intermediate size equals the hybrid's ACTIVE feed-forward width (top * ff + shared ff) so a token costs about the same FLOPs.
@@ -170,6 +171,72 @@ def _goponex_floors(name, t, s_pre, ctx, b, prefill):
     return out
 
 
+# the hyper-connected design at the same width / vocabulary / attention / expert sizes and as many layer RUNS: six layers (chunked,
+# windowed, latent, windowed, chunked, windowed) of which the first two run twice; windowed layers with the narrower values
+NATALORN_MIXERS = {
+    "1b": dict(streams=4, vdim=64, chunk=1024, softcap=30.0, groups=(4, 2)),
+    "small": dict(streams=2, vdim=64, chunk=512, softcap=30.0, groups=(4, 2)),
+}
+
+
+def natalorn_config(name: str):
+    from .hybrid import HybridConfig
+
+    sz, nm, la = SIZES[name], NATALORN_MIXERS[name], KENETAR_MIXERS[name]["latent"]
+    a, m = sz["attn"], sz["moe"]
+    mlp = {"kind": "moe", "router": {"experts": m["experts"], "top": m["top"], "scale": 2.5,
+                                     "groups": {"count": nm["groups"][0], "keep": nm["groups"][1]}},
+           "expert": {"ff": m["ff"]}, "shared": {"ff": m["shared"]}}
+    base = {"heads": a["heads"], "kv_heads": a["kv_heads"], "dim": a["dim"], "scale": a["dim"] ** -0.5}
+    win = {"type": "attention", "mlp": mlp, "mixer": dict(base, vdim=nm["vdim"], mask={"size": a["window"]})}
+    chk = {"type": "attention_2", "mlp": mlp, "mixer": dict(base, vdim=a["vdim"], mask={"size": nm["chunk"]}, softcap=nm["softcap"])}
+    lat = {"type": "latent_attention", "mlp": mlp, "mixer": dict(la, scale=(la["dim"] + la["rot_dim"]) ** -0.5, mask={"size": a["window"]},
+                                                                rot={"dims": la["rot_dim"], "base": 10000.0})}
+    assert sz["layers"] == 8
+    return HybridConfig.from_dict({"architecture": "Natalorn", "vocab": sz["vocab"], "width": sz["width"], "norm": {"eps": 1e-6},
+                                   "streams": nm["streams"], "loop": {"start": 0, "stop": 2, "times": 2},
+                                   "layers": [chk, win, lat, win, chk, win]})
+
+
+def _natalorn_floors(name, t, s_pre, ctx, b, prefill):
+    """Algorithmic (flops, bytes) per launch of the hyper-connected design's own kernels at `t` tokens."""
+    sz, nm, la = SIZES[name], NATALORN_MIXERS[name], KENETAR_MIXERS[name]["latent"]
+    a, m, w, st = sz["attn"], sz["moe"], sz["width"], nm["streams"]
+    h, g, d, win, ck = a["heads"], a["kv_heads"], a["dim"], a["window"], nm["chunk"]
+
+    def att(seen, heads, kv_bytes, dk, dv):  # seen(i): keys that position i sees
+        pairs = float(sum(seen(i) for i in range(s_pre))) if prefill else float(b * seen(ctx))
+        rows = s_pre if prefill else b * seen(ctx)
+        return 2.0 * heads * pairs * (dk + dv), rows * kv_bytes + t * heads * (4.0 * dk + 2.0 * dv)
+
+    wnd = att(lambda i: min(i + 1, win), h, 2.0 * g * (d + nm["vdim"]), d, nm["vdim"])
+    chk = att(lambda i: i % ck + 1, h, 2.0 * g * (d + a["vdim"]), d, a["vdim"])
+    row = la["kv_rank"] + la["rot_dim"]
+    lat = att(lambda i: min(i + 1, win), la["heads"], 2.0 * row, row, la["kv_rank"])
+    pairs = t * m["top"]
+    used = min(m["experts"], pairs)
+    out = {}
+    for kern in ("swa_sink_attn_prefill", "swa_sink_attn_prefill_tc", "swa_sink_attn", "swa_sink_attn_decode_tc"):
+        out.update({kern: wnd, kern + "[chunk+cap]": chk, kern + "[latent]": lat})
+    out.update({
+        "latent_attn_decode": lat,
+        "hyper_residual": (2.0 * t * w * st * (st + 2), t * w * (8.0 * st + 4 + 2)),
+        "hyper_residual[experts]": (2.0 * t * w * st * (st + 2), t * w * (8.0 * st + 4 + 4.0 * m["top"] + 2)),
+        "hyper_embed": (0.0, t * w * (2.0 + 4 * st + 2)),
+        "moe_topk_grouped": (0.0, t * 4.0 * (m["experts"] + 2 * m["top"])),
+        "moe_gate_up_glu": (4.0 * pairs * m["ff"] * w, used * 4.0 * m["ff"] * w + t * 2 * w + pairs * 2 * m["ff"]),
+        "moe_down": (2.0 * pairs * m["ff"] * w, used * 2.0 * m["ff"] * w + pairs * (2 * m["ff"] + 4 * w)),
+        "moe_gather_scale": (0.0, pairs * w * 4.0),
+        "kv_write_vmix": (0.0, t * g * (d + nm["vdim"]) * 6.0),
+        "qk_norm_rope_kv_write": (0.0, t * (8.0 * h * d + 6.0 * g * (d + a["vdim"]))),
+        "latent_kv_write": (0.0, t * row * 6.0),
+        "latent_q_prep": (0.0, t * la["heads"] * ((la["dim"] + la["rot_dim"]) * 4 + la["dim"] * 2 + la["rot_dim"] * 4.0)),
+        "rmsnorm_cols": (0.0, t * la["q_rank"] * 6.0),
+        "glu": (0.0, t * m["shared"] * 10.0),
+    })
+    return out
+
+
 def zudarax_config(name: str):
     from .hybrid import HybridConfig
 
@@ -247,7 +314,7 @@ def _kenetar_floors(name, t, keys_per_query, kv_tokens, nseq):
     att = (2.0 * t * la["heads"] * keys_per_query * (row + la["kv_rank"]),
            2.0 * kv_tokens * row + t * la["heads"] * (4 * row + 2 * la["kv_rank"]))
     return {
-        "swa_sink_attn_prefill": att, "swa_sink_attn": att, "latent_attn_decode": att,
+        "swa_sink_attn_prefill[latent]": att, "swa_sink_attn[latent]": att, "latent_attn_decode": att,
         "delta_scan": (8.0 * t * d["heads"] * d["dim"] * d["vdim"],
                        t * (4 * c + 4 * hp) + 8.0 * nseq * d["heads"] * d["dim"] * d["vdim"]),
         "delta_prep": (0.0, t * 16.0 * d["kv_heads"] * d["dim"]),
@@ -401,6 +468,10 @@ def _time_hybrid(cfg, sz, args, floors_fn, flush, hbm, peak):
     return out, rows, nblocks, mml, ptoks, dtoks
 
 
+# design -> the models it is timed beside (the others: the dense decoder)
+BESIDE = {"kenetar": ("pumopel",), "gerupel": ("pumopel",), "goponex": ("gerupel", "pumopel"), "natalorn": ("kenetar", "zudarax", "pumopel")}
+
+
 def run(args):
     from .model import B200CausalLM
 
@@ -410,52 +481,42 @@ def run(args):
     flush = torch.empty(192 << 20, dtype=torch.float32, device=dev)  # 768 MB > L2
     names = list(SIZES) if args.hybrid == "all" else [args.hybrid]
     for name in names:
-        kenetar, zudarax, gerupel = name.startswith("kenetar-"), name.startswith("zudarax-"), name.startswith("gerupel-")
-        goponex = name.startswith("goponex-")
-        short = name.split("-", 1)[1] if kenetar or zudarax or gerupel or goponex else name
+        design, _, short = name.rpartition("-")
         sz = SIZES[short]
-        cfg = hybrid_config(sz)
         s_pre, b, ctx = sz["prefill"], sz["batch"], sz["ctx"]
         bs = 32
-        res = {"metric": "goponex_vs_gerupel_tokens_per_s" if goponex else "gerupel_vs_pumopel_tokens_per_s" if gerupel else "kenetar_vs_pumopel_tokens_per_s" if kenetar else "zudarax_vs_dense_tokens_per_s" if zudarax else
-               "hybrid_vs_dense_tokens_per_s", "size": name,
+        beside = BESIDE.get(design)
+        metric = f"{design}_vs_{beside[0]}" if beside else "zudarax_vs_dense" if design else "hybrid_vs_dense"
+        res = {"metric": metric + "_tokens_per_s", "size": name,
                "dtype": "bf16", "data": "synthetic (random weights)",
                "roofline_peaks": {"hbm_gbs": hbm / 1e9, "bf16_tflops": peak / 1e12, "source": src},
                "config": {"width": sz["width"], "layers": sz["layers"], "prefill_tokens": s_pre, "decode_batch": b,
                           "decode_ctx": ctx, "l2": "flushed between timed steps"}}
         win = sz["attn"]["window"]
-        pum_floors = lambda t, pre: _floors(cfg, sz, t, min(win, s_pre / 2) if pre else min(win, ctx + 1),  # noqa: E731
-                                            s_pre if pre else b * min(win, ctx + 1), 1 if pre else b)
-        if goponex:
-            gop_floors = lambda t, pre: _goponex_floors(short, t, s_pre, ctx, b, pre)  # noqa: E731
-            ger_floors = lambda t, pre: _gerupel_floors(short, t, s_pre, ctx, b, pre)  # noqa: E731
-            res["goponex"] = _time_hybrid(goponex_config(short), sz, args, gop_floors, flush, hbm, peak)[0]
-            res["gerupel"] = _time_hybrid(gerupel_config(short), sz, args, ger_floors, flush, hbm, peak)[0]
-            res["pumopel"] = _time_hybrid(cfg, sz, args, pum_floors, flush, hbm, peak)[0]
-            res["gpu_launches"] = ops.launch_count()
-            print(json.dumps(res), flush=True)
-            continue
-        if gerupel:
-            ger_floors = lambda t, pre: _gerupel_floors(short, t, s_pre, ctx, b, pre)  # noqa: E731
-            res["gerupel"] = _time_hybrid(gerupel_config(short), sz, args, ger_floors, flush, hbm, peak)[0]
-            res["pumopel"] = _time_hybrid(cfg, sz, args, pum_floors, flush, hbm, peak)[0]
-            res["gpu_launches"] = ops.launch_count()
-            print(json.dumps(res), flush=True)
-            continue
-        if kenetar:
-            ken_floors = lambda t, pre: _kenetar_floors(short, t, s_pre / 2 if pre else ctx + 1,  # noqa: E731
-                                                        s_pre if pre else b * (ctx + 1), 1 if pre else b)
-            res["kenetar"] = _time_hybrid(kenetar_config(short), sz, args, ken_floors, flush, hbm, peak)[0]
-            res["pumopel"] = _time_hybrid(cfg, sz, args, pum_floors, flush, hbm, peak)[0]
+        models = {  # design -> (configuration, (flops, bytes) of its kernels)
+            "pumopel": (lambda: hybrid_config(sz), lambda t, pre: _floors(None, sz, t, min(win, s_pre / 2) if pre else min(win, ctx + 1),
+                                                                          s_pre if pre else b * min(win, ctx + 1), 1 if pre else b)),
+            "kenetar": (lambda: kenetar_config(short), lambda t, pre: _kenetar_floors(short, t, s_pre / 2 if pre else ctx + 1,
+                                                                                      s_pre if pre else b * (ctx + 1), 1 if pre else b)),
+            "zudarax": (lambda: zudarax_config(short), lambda t, pre: _zudarax_floors(short, t, s_pre, ctx, b, pre)),
+            "gerupel": (lambda: gerupel_config(short), lambda t, pre: _gerupel_floors(short, t, s_pre, ctx, b, pre)),
+            "goponex": (lambda: goponex_config(short), lambda t, pre: _goponex_floors(short, t, s_pre, ctx, b, pre)),
+            "natalorn": (lambda: natalorn_config(short), lambda t, pre: _natalorn_floors(short, t, s_pre, ctx, b, pre)),
+        }
+
+        def timed(which):
+            config, floors = models[which]
+            return _time_hybrid(config(), sz, args, floors, flush, hbm, peak)
+
+        if beside:
+            for which in (design, *beside):
+                res[which] = timed(which)[0]
             res["gpu_launches"] = ops.launch_count()
             print(json.dumps(res), flush=True)
             continue
         # ---------------- hybrid
-        if zudarax:
-            zud_floors = lambda t, pre: _zudarax_floors(short, t, s_pre, ctx, b, pre)  # noqa: E731
-            res["zudarax"], rows, nblocks, mml, ptoks, dtoks = _time_hybrid(zudarax_config(short), sz, args, zud_floors, flush, hbm, peak)
-        else:
-            res["hybrid"], rows, nblocks, mml, ptoks, dtoks = _time_hybrid(cfg, sz, args, pum_floors, flush, hbm, peak)
+        which = design or "pumopel"
+        res[design or "hybrid"], rows, nblocks, mml, ptoks, dtoks = timed(which)
         per = -(-mml // bs)
         # ---------------- dense decoder of equal size
         shape = dense_shape(sz)
